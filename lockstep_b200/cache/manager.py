@@ -5,7 +5,8 @@ Layers are sorted into groups by what their mixer declares (``CacheNeed``):
   block table per request; layers that read all keys and layers that read a
   window of them are different groups with pages of their own; a windowed
   group gives a page back as soon as every position in it lies behind the
-  window;
+  window (but the pages of the first positions that stay visible, where a need
+  names such);
 - a state group keeps one tensor of fixed size per request in a slot.
 A live request owns one slot id; it is its row in every group's block table
 and its index in every state tensor.  Pages are handed out lowest-first,
@@ -57,6 +58,8 @@ class PagedGroup:
                  poison_freed_pages: bool = False):
         self.need, self.entries = need, list(entries)
         self.page_size, self.window = int(page_size), int(need.window)
+        # leading pages that are kept although the window has passed them
+        self.kept_pages = -(-int(need.keep_first) // self.page_size) if self.window else 0
         self.allocator = PageAllocator(num_pages)
         self.max_pages_per_seq = int(max_pages_per_seq)
         # One row and one page more than requests can hold: the padding row (index max_live) maps
@@ -114,6 +117,10 @@ class PagedGroup:
         lo = q - self.window + 1
         return max(0, lo) // self.page_size
 
+    def readable(self, logical: int, pos: int) -> bool:
+        """Whether a query at position ``pos`` or a later one can still read logical page ``logical``."""
+        return logical < self.kept_pages or logical >= self.first_needed_page(pos)
+
     def pages_short(self, uid: str, total_tokens: int) -> int:
         """How many new pages ``reserve(uid, total_tokens)`` would take."""
         seq = self.seqs[uid]
@@ -141,7 +148,7 @@ class PagedGroup:
         first = self.first_needed_page(kv_len // self.page_size * self.page_size if self.keep_boundary_window
                                        else kv_len)
         freed = 0
-        for logical in range(min(first, len(seq.pages))):
+        for logical in range(min(self.kept_pages, len(seq.pages)), min(first, len(seq.pages))):
             page = seq.pages[logical]
             if page >= 0:
                 self._give_back(page)
@@ -323,7 +330,8 @@ class CacheManager:
         for g in self.paged:
             need = -(-total_tokens // self.page_size)
             if g.window and total_tokens > max_portion:
-                need = min(need, -(-(g.window - 1 + max_portion) // self.page_size) + 1 + g.keep_boundary_window)
+                need = min(need, -(-(g.window - 1 + max_portion) // self.page_size) + 1 + g.keep_boundary_window
+                           + g.kept_pages)
             worst = max(worst, need)
         return worst
 

@@ -11,8 +11,9 @@ page of tokens and names the page that holds them in each group, or -1 where the
 request had already given that page back (it lay behind a window).  A prefix of
 n pages can be adopted if every group still has the pages that the first new
 token can read: all n where every key is kept, those that reach into the window
-of position n x page_size elsewhere.  ``lookup`` returns the longest such prefix,
-with -1 in a group's list for the pages that group does not need.  So a model with
+of position n x page_size elsewhere (and those of the first positions, where these
+stay visible).  ``lookup`` returns the longest such prefix, with -1 in a group's
+list for the pages that group does not need.  So a model with
 windowed layers reuses a prefix where its window's pages were kept (the end of a
 finished request's context: the next turn of the same conversation), and one
 without windows reuses any shared prefix.  A fixed-size state cannot be shared by
@@ -95,9 +96,8 @@ class PrefixIndex:
         if limit is not None:
             n = min(n, limit // self.page_size)
         while n > 0:
-            first = [g.first_needed_page(n * self.page_size) for g in groups]
             if all(found[i] is not None and found[i].pages[gi] >= 0
-                   for gi in range(len(groups)) for i in range(first[gi], n)):
+                   for gi, g in enumerate(groups) for i in range(n) if g.readable(i, n * self.page_size)):
                 break
             n -= 1
         if n == 0:
@@ -106,9 +106,8 @@ class PrefixIndex:
             if e is not None:
                 e.hits += 1
         self.stats["hit_pages"] += n
-        first = [g.first_needed_page(n * self.page_size) for g in groups]
-        return n * self.page_size, [[found[i].pages[gi] if i >= first[gi] else -1 for i in range(n)]
-                                    for gi in range(len(groups))]
+        return n * self.page_size, [[found[i].pages[gi] if g.readable(i, n * self.page_size) else -1 for i in range(n)]
+                                    for gi, g in enumerate(groups)]
 
     def insert(self, tokens, groups, uid: str) -> int:
         """Index the whole pages of ``tokens`` that request ``uid`` holds; returns how many

@@ -13,9 +13,11 @@ from . import kemirax as _kemirax  # registers Kemirax
 from .kemirax import KemiraxConfig
 from . import pikurax as _pikurax  # registers Pikurax
 from .pikurax import PikuraxConfig
+from . import kusolorn as _kusolorn  # registers Kusolorn
+from .kusolorn import KusolornConfig
 
 __all__ = [
-    "ConfigError", "KemiraxConfig", "LayerRun", "LayerSpec", "MalazenConfig", "ModelSpec", "PartSpec", "PikuraxConfig", "Qwen3Config", "SevipelConfig",
+    "ConfigError", "KemiraxConfig", "KusolornConfig", "LayerRun", "LayerSpec", "MalazenConfig", "ModelSpec", "PartSpec", "PikuraxConfig", "Qwen3Config", "SevipelConfig",
     "architecture_name", "config_from_dict", "known_architectures", "load_config",
     "own_tensors", "register_architecture", "tensor_name", "unregister_architecture",
 ]

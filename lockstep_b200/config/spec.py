@@ -104,9 +104,13 @@ class ModelSpec:
     # a part that mixes the embedding's output into the residual stream where the schedule says so
     # (``LayerRun.inject``); its tensors lie under ``names["injection"]``
     injection: PartSpec | None = None
+    # parts of category "table" that several layers use, by the name the layers' parts ask for them under (in
+    # ``Runtime.shared``); the tensors of part ``x`` lie under ``names["x"]``
+    shared: Mapping[str, PartSpec] = field(default_factory=dict)
 
     def __post_init__(self):
         object.__setattr__(self, "names", _freeze(self.names))
+        object.__setattr__(self, "shared", _freeze(self.shared))
         object.__setattr__(self, "layers", tuple(self.layers))
         object.__setattr__(self, "schedule", tuple(self.schedule))
         object.__setattr__(self, "optional_tensors", tuple(self.optional_tensors))

@@ -50,8 +50,8 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
                             float* __restrict__ part_acc, float* __restrict__ part_ml,
                             const int* __restrict__ work, const int* __restrict__ block_table,
                             int table_stride, int nq, int nkv, int page_size, int num_pages, int window,
-                            float scale, const float* __restrict__ slopes, const float* __restrict__ log_rates,
-                            int* err) {
+                            int keep_first, float scale, float softcap, const float* __restrict__ slopes,
+                            const float* __restrict__ log_rates, int* err) {
   // The work list, the block table and every key older than this step's token are there
   // before the step's first kernel starts, so the first chunks are fetched while the kernel
   // before this one (which writes the token's own key and value, and q) still runs.
@@ -120,10 +120,11 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
     const int i = lane >> 2, b = lane & 3;
     if (i < n_iter && b < boxes) {
       const int c0 = s_lo + (i * WARPS + warp) * CHUNK;
-      if (c0 < s_hi && c0 + CHUNK > row_lo) {
+      if (c0 < s_hi && (c0 + CHUNK > row_lo || c0 < keep_first)) {
         int key = c0 + b * rows_per_box;
         if (key >= s_hi) key = s_hi - 1;          // beyond the split's end: any page that exists
-        if (key < row_lo) key = row_lo;           // behind the window: pages may have been given back
+        if (key >= keep_first && key < row_lo && key / page_size != row_lo / page_size)
+          key = keep_first > 0 ? 0 : row_lo;      // behind the window: pages may have been given back
         my_page = table_row[key / page_size];
         if (my_page < 0 || my_page >= num_pages) {
           ls_record_fault(err, LS_DEV_PAGE_RANGE, key);
@@ -158,7 +159,7 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
   auto chunk_start = [&](int i) { return s_lo + (i * WARPS + warp) * CHUNK; };
   auto chunk_live = [&](int i) {
     const int c0 = chunk_start(i);
-    return i < n_iter && c0 < s_hi && c0 + CHUNK > row_lo;
+    return i < n_iter && c0 < s_hi && (c0 + CHUNK > row_lo || c0 < keep_first);
   };
 
   int it = 0;
@@ -232,11 +233,11 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = c0 + nt * 8 + cq + (e & 1);
-        const bool keep = key < s_hi && key >= row_lo;
+        const bool keep = key < s_hi && ls_sees(key, row_lo, keep_first);
         // (log_rates: slopes[head] x ln(1 + log_rates[head] x distance) is taken off the score)
         s[nt][e] = !keep ? -CUDART_INF_F
                    : log_rates != nullptr ? s[nt][e] * scale - bias_a[e >> 1] * log1pf(bias_b[e >> 1] * (float)(pos - key))
-                                          : s[nt][e] * scale;
+                                          : ls_capped(s[nt][e] * scale, softcap);
         tile_max[e >> 1] = fmaxf(tile_max[e >> 1], s[nt][e]);
       }
     float alpha[2];
@@ -283,11 +284,11 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
     // Values of masked keys (past the row's last key, behind its window) are whatever
     // the page holds; their weight is 0, but 0 * inf is not: clear those rows.
     {
-      const int valid_hi = s_hi - c0, valid_lo = row_lo - c0;
+      const int valid_hi = s_hi - c0, valid_lo = row_lo - c0, valid_kept = keep_first - c0;
       if (valid_hi < CHUNK || valid_lo > 0) {
         for (int idx = lane; idx < HALVES * CHUNK * 8; idx += 32) {
           const int half = idx / (CHUNK * 8), key = (idx / 8) % CHUNK, ch = idx & 7;
-          if (key >= valid_hi || key < valid_lo)
+          if (key >= valid_hi || (key < valid_lo && key >= valid_kept))
             *reinterpret_cast<uint4*>(aligned + (v_smem - base) + half * HALF_BYTES + key * 128 + ch * 16) =
                 make_uint4(0u, 0u, 0u, 0u);
         }
@@ -383,8 +384,8 @@ EncodeTiled encode_fn() {
 template <int HALVES>
 int launch(const CUtensorMap& map, const void* q, float* part_acc, float* part_ml, const int* work,
            int n_work, const int* block_table, int table_stride, int nq, int nkv, int page_size,
-           int num_pages, int window, float scale, const float* slopes, const float* log_rates, int* err,
-           cudaStream_t stream) {
+           int num_pages, int window, int keep_first, float scale, float softcap, const float* slopes,
+           const float* log_rates, int* err, cudaStream_t stream) {
   const size_t smem = (size_t)WARPS * 2 * HALVES * CHUNK * 128 + 128 + 16 * HALVES * 128 + 1024;
   static bool configured = false;
   if (!configured) {
@@ -396,7 +397,7 @@ int launch(const CUtensorMap& map, const void* q, float* part_acc, float* part_m
   dim3 grid(n_work, nkv);
   LS_COUNT(LS_K_ATTENTION_DECODE_MMA), ls_launch(attention_decode_mma_kernel<HALVES>, grid, WARPS * 32, smem, stream, 
       map, (const __nv_bfloat16*)q, part_acc, part_ml, work, block_table, table_stride, nq, nkv, page_size,
-      num_pages, window, scale, slopes, log_rates, err);
+      num_pages, window, keep_first, scale, softcap, slopes, log_rates, err);
   return ls_launch_status();
 }
 
@@ -407,9 +408,11 @@ int launch(const CUtensorMap& map, const void* q, float* part_acc, float* part_m
 LS_API int ls_attention_decode_mma(const void* q, const void* pages, float* part_acc, float* part_ml,
                                    const int* work, int n_work, const int* block_table,
                                    int table_stride, int nq, int nkv, int d, int page_size,
-                                   int num_pages, int window, float scale, const float* slopes,
-                                   const float* log_rates, int* err, cudaStream_t stream) {
+                                   int num_pages, int window, int keep_first, float scale,
+                                   float softcap, const float* slopes, const float* log_rates, int* err,
+                                   cudaStream_t stream) {
   if (n_work <= 0) return 0;
+  if (keep_first < 0 || (softcap > 0.f && log_rates != nullptr)) return LS_E_SIZE;
   if ((slopes != nullptr) != (log_rates != nullptr)) return LS_E_SIZE;      // a linear bias alone: the CUDA-core kernels
   if (nq <= 0 || nkv <= 0 || nq % nkv || nq / nkv > 16 || nkv > 65535) return LS_E_SIZE;
   if (d != 64 && d != 128) return LS_E_SIZE;
@@ -429,9 +432,9 @@ LS_API int ls_attention_decode_mma(const void* q, const void* pages, float* part
     return LS_E_SIZE;
   if (d == 64)
     return launch<1>(map, q, part_acc, part_ml, work, n_work, block_table, table_stride, nq, nkv, page_size,
-                     num_pages, window, scale, slopes, log_rates, err, stream);
+                     num_pages, window, keep_first, scale, softcap, slopes, log_rates, err, stream);
   return launch<2>(map, q, part_acc, part_ml, work, n_work, block_table, table_stride, nq, nkv, page_size,
-                   num_pages, window, scale, slopes, log_rates, err, stream);
+                   num_pages, window, keep_first, scale, softcap, slopes, log_rates, err, stream);
 }
 
 LS_API const char* ls_constants_attention_decode_mma() {

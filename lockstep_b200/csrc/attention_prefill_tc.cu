@@ -154,6 +154,9 @@ struct Item {
   const int* table_row;
   int tok0, ntok, pos0, h, kvh;
   int pos_last, key_lo, tile_first, n_tiles;
+  int lead;                  // tiles 0 .. lead - 1 come before tile_first (first keys that stay visible)
+  // the place among all tiles of 128 keys of this item's tile `it`
+  __device__ __forceinline__ int tile(int it) const { return it < lead ? it : tile_first + it - lead; }
 };
 
 // HALVES = d / 64.  Shared memory: Q [HALVES][128 rows][128 B]; two stages of K and of V
@@ -170,13 +173,14 @@ struct Item {
 // slopes[head] x lg2(1 + log_rates[head] x distance), one more special-function instruction a score),
 // and the softmax's denominator one more term exp(sinks[head]) at the end of a row.  With slopes and no log_rates the
 // bias is slopes[head] x distance, and with cap_log2 > 0 (a cap times lg2 e) the scaled score first becomes
-// cap tanh(score / cap): one tanh.approx a score, again in the units of the exponentials.
+// cap tanh(score / cap): one tanh.approx a score, again in the units of the exponentials.  keep_first > 0: the first
+// keep_first keys of the sequence stay visible behind the window; their tiles come first.
 template <int HALVES, bool EXTRAS>
 __global__ void __launch_bounds__(THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                             __nv_bfloat16* __restrict__ out, const int* __restrict__ work, int n_work,
                             const int* __restrict__ block_table, int table_stride, int nq, int nkv, int page_size,
-                            int num_pages, int window, float scale_log2, const float* __restrict__ slopes,
+                            int num_pages, int window, int keep_first, float scale_log2, const float* __restrict__ slopes,
                             const float* __restrict__ log_rates, const float* __restrict__ sinks, float cap_log2, int* err) {
   ls_dependency_trigger();
   constexpr int D = HALVES * 64;
@@ -210,6 +214,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int total_items = n_work * nq;
   const int blocks = (int)gridDim.x;
+  const int kept = EXTRAS ? keep_first : 0;
 
   // the item of this block in round `round`: 0 none is left, 1 an item, 2 a padding item (nothing to do)
   auto get_item = [&](int round, Item& I) -> int {
@@ -227,7 +232,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     I.pos_last = I.pos0 + I.ntok - 1;
     I.key_lo = ls_first_key(I.pos0, window);   // first key any row reads
     I.tile_first = I.key_lo / BLOCK_N;
-    I.n_tiles = I.pos_last / BLOCK_N + 1 - I.tile_first;
+    I.lead = kept > 0 ? min((kept + BLOCK_N - 1) / BLOCK_N, I.tile_first) : 0;
+    I.n_tiles = I.pos_last / BLOCK_N + 1 - I.tile_first + I.lead;
     return 1;
   };
 
@@ -237,9 +243,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   auto lookup = [&](const Item& I, int it) {
     int page = 0;
     if (it < I.n_tiles && lane < boxes) {
-      int key = (I.tile_first + it) * BLOCK_N + lane * rows_per_box;
+      int key = I.tile(it) * BLOCK_N + lane * rows_per_box;
       if (key > I.pos_last) key = I.pos_last;            // past the last key: any page that exists
-      if (key < I.key_lo) key = I.key_lo;                // behind the window: pages may have been given back
+      if (key >= kept && key < I.key_lo && key / page_size != I.key_lo / page_size)
+        key = kept > 0 ? 0 : I.key_lo;                   // behind the window: pages may have been given back
       page = I.table_row[key / page_size];               // checked where it is used: the load stays in flight
     }
     return page;
@@ -310,7 +317,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int g = gt + it;
         const int s = g & 1;
         const uint32_t phase = (uint32_t)(g >> 1) & 1u;
-        const int c0 = (I.tile_first + it) * BLOCK_N;
+        const int c0 = I.tile(it) * BLOCK_N;
         ok = *failed == 0 && mbar_wait(&free_bar[s], phase ^ 1u);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) {
@@ -429,7 +436,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       const int kind = get_item(round, I);
       if (kind == 0) break;
       if (kind == 2) continue;
-      const int pos0 = I.pos0, pos_last = I.pos_last, tile_first = I.tile_first, n_tiles = I.n_tiles;
+      const int pos0 = I.pos0, pos_last = I.pos_last, n_tiles = I.n_tiles;
       const int pos = pos0 + row;
       const int lo = ls_first_key(pos, window);
       const int lo_last = ls_first_key(pos_last, window);
@@ -452,7 +459,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       for (int it = 0; it < n_tiles; ++it) {
         const int g = gt + it;
         const int s = g & 1;
-        const int c0 = (tile_first + it) * BLOCK_N + group * HC;     // first key of this thread
+        const int t0 = I.tile(it) * BLOCK_N;                         // first key of the tile
+        const int c0 = t0 + group * HC;                              // first key of this thread
         if (ok && !mbar_wait(&s_full[s], (uint32_t)(g >> 1) & 1u)) ok = false;
         fence_after_sync();
         // this thread's scores into registers; the buffer is free once all have theirs
@@ -481,7 +489,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           }
         }
         // every key of the tile is seen by every row: no masks (uniform over the block)
-        const bool full_tile = (tile_first + it) * BLOCK_N + BLOCK_N - 1 <= pos0 && (tile_first + it) * BLOCK_N >= lo_last;
+        const bool full_tile = t0 + BLOCK_N - 1 <= pos0 && (t0 >= lo_last || t0 + BLOCK_N <= kept);
         float mx[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
         if (full_tile) {
 #pragma unroll
@@ -491,7 +499,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           // selects, not branches: a masked score counts as -inf
 #pragma unroll
           for (int jj = 0; jj < HC; ++jj) {
-            const bool keep = (c0 + jj <= pos) & (c0 + jj >= lo);
+            const bool keep = (c0 + jj <= pos) & ((c0 + jj >= lo) | (EXTRAS && c0 + jj < kept));
             mx[jj & 3] = fmaxf(mx[jj & 3], keep ? __uint_as_float(sc[jj]) : -CUDART_INF_F);
           }
         }
@@ -547,7 +555,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
               for (int jj = 0; jj < 8; ++jj) {
                 const int key = c0 + n0 + jj;
-                const bool keep = (key <= pos) & (key >= lo) & !dead;
+                const bool keep = (key <= pos) & ((key >= lo) | (EXTRAS && key < kept)) & !dead;
                 p[jj] = ex2(keep ? fmaf(__uint_as_float(sc[n0 + jj]), scale_eff, neg_m) : -CUDART_INF_F);
               }
             }
@@ -563,9 +571,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const float psum = (ps[0] + ps[1]) + (ps[2] + ps[3]);
         // value rows of keys past the last position were never written: they must not be NaN,
         // since P is zero there and the MMA multiplies all the same
-        if ((tile_first + it) * BLOCK_N + BLOCK_N - 1 > pos_last) {
+        if (t0 + BLOCK_N - 1 > pos_last) {
           if (ok && !mbar_wait(&v_full[s], (uint32_t)(g >> 1) & 1u)) ok = false;
-          if (ok && group < HALVES && (tile_first + it) * BLOCK_N + row > pos_last) {
+          if (ok && group < HALVES && t0 + row > pos_last) {
             uint4* vrow = reinterpret_cast<uint4*>(v_ptr + s * KV_BYTES + group * HALF_BYTES + row * 128);
 #pragma unroll
             for (int q8 = 0; q8 < 8; ++q8) vrow[q8] = make_uint4(0u, 0u, 0u, 0u);
@@ -1128,8 +1136,8 @@ int pair_heads = 1;
 template <int HALVES>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, void* out, const int* work, int n_work,
            const int* block_table, int table_stride, int nq, int nkv, int page_size, int num_pages, int window,
-           float scale, const float* slopes, const float* log_rates, const float* sinks, float softcap, int* err,
-           cudaStream_t stream) {
+           int keep_first, float scale, const float* slopes, const float* log_rates, const float* sinks, float softcap,
+           int* err, cudaStream_t stream) {
   constexpr int KV_BYTES = HALVES * HALF_BYTES;
   const size_t smem = (size_t)KV_BYTES * (1 + 2 * STAGES) + 256 + 3 * 128 * GROUPS * 4 + 1024;
   static bool configured = false;
@@ -1141,13 +1149,13 @@ int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, void* out, const
       return LS_E_SMEM;
     configured = true;
   }
-  if (slopes != nullptr || sinks != nullptr || softcap > 0.f) {
-    // a bias on the scores or a sink: the kernel with a head a block knows them
+  if (slopes != nullptr || sinks != nullptr || softcap > 0.f || keep_first > 0) {
+    // a bias on the scores, a cap, a sink or kept first keys: the kernel with a head a block knows them
     const long long items = (long long)n_work * nq;
     const int blocks = items < sm_count() ? (int)items : sm_count();
     LS_COUNT(LS_K_ATTENTION_PREFILL_TC), ls_launch(attention_prefill_tc_kernel<HALVES, true>, dim3(blocks), THREADS, smem, stream, map_q, map_kv,
               (__nv_bfloat16*)out, work, n_work, block_table, table_stride, nq, nkv, page_size, num_pages, window,
-              scale * 1.4426950408889634f, slopes, log_rates, sinks, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, err);
+              keep_first, scale * 1.4426950408889634f, slopes, log_rates, sinks, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, err);
     return ls_launch_status();
   }
   // two heads of a key head in a block where the group size is even and there are items enough
@@ -1174,7 +1182,7 @@ int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, void* out, const
   const long long items = (long long)n_work * nq;
   const int blocks = items < sm_count() ? (int)items : sm_count();
   LS_COUNT(LS_K_ATTENTION_PREFILL_TC), ls_launch(attention_prefill_tc_kernel<HALVES, false>, dim3(blocks), THREADS, smem, stream, map_q, map_kv, (__nv_bfloat16*)out, work, n_work,
-            block_table, table_stride, nq, nkv, page_size, num_pages, window, scale * 1.4426950408889634f,
+            block_table, table_stride, nq, nkv, page_size, num_pages, window, 0, scale * 1.4426950408889634f,
             (const float*)nullptr, (const float*)nullptr, (const float*)nullptr, 0.f, err);
   return ls_launch_status();
 }
@@ -1190,9 +1198,11 @@ LS_API void ls_set_attention_prefill_pairs(int mode) { pair_heads = mode < 0 ? 0
 // launched nothing.
 LS_API int ls_attention_prefill_tc(const void* q, const void* pages, void* out, int tokens, const int* work,
                                    int n_work, const int* block_table, int table_stride, int nq, int nkv, int d,
-                                   int page_size, int num_pages, int window, float scale, const float* slopes,
-                                   const float* log_rates, const float* sinks, float softcap, int* err, cudaStream_t stream) {
+                                   int page_size, int num_pages, int window, int keep_first, float scale,
+                                   const float* slopes, const float* log_rates, const float* sinks, float softcap,
+                                   int* err, cudaStream_t stream) {
   if (n_work <= 0 || tokens <= 0) return 0;
+  if (keep_first < 0) return LS_E_SIZE;
   if (log_rates != nullptr && (slopes == nullptr || softcap > 0.f)) return LS_E_SIZE;
   if (nq <= 0 || nkv <= 0 || nq % nkv || n_work > 65535) return LS_E_SIZE;
   if (d != 64 && d != 128) return LS_E_SIZE;
@@ -1205,9 +1215,9 @@ LS_API int ls_attention_prefill_tc(const void* q, const void* pages, void* out, 
   if (!encode(&map_kv, pages, (uint64_t)d, (uint64_t)rows, page_size < BLOCK_N ? page_size : BLOCK_N)) return LS_E_SIZE;
   if (d == 64)
     return launch<1>(map_q, map_kv, out, work, n_work, block_table, table_stride, nq, nkv, page_size, num_pages,
-                     window, scale, slopes, log_rates, sinks, softcap, err, stream);
+                     window, keep_first, scale, slopes, log_rates, sinks, softcap, err, stream);
   return launch<2>(map_q, map_kv, out, work, n_work, block_table, table_stride, nq, nkv, page_size, num_pages,
-                   window, scale, slopes, log_rates, sinks, softcap, err, stream);
+                   window, keep_first, scale, slopes, log_rates, sinks, softcap, err, stream);
 }
 
 LS_API const char* ls_constants_attention_prefill_tc() {

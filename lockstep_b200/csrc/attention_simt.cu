@@ -17,7 +17,9 @@
 // pages: [num_pages, 2, nkv, page_size, d]; q, out: [tokens, nq, d].
 // work item (8 ints): request row in the block table, first token (packed
 // index), number of tokens, position of the first token, first split, end
-// split, first scratch slot (-1: serial, write `out`), unused.
+// split, first scratch slot (-1: serial, write `out`), leading splits (serial:
+// splits 0 .. n - 1 are walked before the first split, for the sake of the
+// first keys of the sequence that stay visible behind a window).
 #include <math_constants.h>
 
 #include "attention_fold.cuh"
@@ -55,7 +57,7 @@ attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ pages, T* _
                       float* __restrict__ part_acc, float* __restrict__ part_ml,
                       const int* __restrict__ work, const int* __restrict__ block_table,
                       int table_stride, int nq, int nkv, int d, int page_size, int num_pages,
-                      int window, float scale, float softcap, const float* __restrict__ slopes,
+                      int window, int keep_first, float scale, float softcap, const float* __restrict__ slopes,
                       const float* __restrict__ log_rates, const float* __restrict__ sinks, int hb, int* err) {
   ls_dependency_sync();
   extern __shared__ __align__(16) float smem[];
@@ -71,7 +73,7 @@ attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ pages, T* _
   const int* w = work + (int64_t)blockIdx.x * 8;
   const int req_row = w[0], tok0 = w[1], ntok = w[2], pos0 = w[3];
   if (ntok == 0) return;                     // padding item of a recorded launch
-  const int split_begin = w[4], split_end = w[5], slot_base = w[6];
+  const int split_begin = w[4], split_end = w[5], slot_base = w[6], leading = w[7];
   const int kvh = ((int)blockIdx.y * hb) / (nq / nkv);
   const int heads_at_once = ntok * hb <= TILE_M ? hb : 1;      // heads that share the tile's rows
   const int tid = threadIdx.x;
@@ -115,7 +117,8 @@ attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ pages, T* _
   for (int j = 0; j < MAX_D / 8; ++j) acc_run[j] = 0.f;
   float m_run = -CUDART_INF_F, l_run = 0.f;
 
-  for (int split = split_begin; split < split_end; ++split) {
+  for (int turn = split_begin - leading; turn < split_end; ++turn) {
+    const int split = turn < split_begin ? turn - (split_begin - leading) : turn;
     const int s_lo = split * LS_SPLIT;
     int s_hi = s_lo + LS_SPLIT;                 // exclusive
     if (s_hi > pos_last + 1) s_hi = pos_last + 1;
@@ -124,10 +127,11 @@ attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ pages, T* _
     float m_s = -CUDART_INF_F, l_s = 0.f;
 
     // tiles lie at fixed offsets from the split's start; those wholly before
-    // the first row's window change nothing and are skipped
+    // the first row's window (and behind the kept first keys) change nothing and are skipped
     int t_first = s_lo;
-    if (key_lo_tile > s_lo) t_first = s_lo + ((key_lo_tile - s_lo) / TILE_N) * TILE_N;
+    if (key_lo_tile > s_lo && s_lo >= keep_first) t_first = s_lo + ((key_lo_tile - s_lo) / TILE_N) * TILE_N;
     for (int n0 = t_first; n0 < s_hi; n0 += TILE_N) {
+      if (n0 >= keep_first && n0 + TILE_N <= key_lo_tile) continue;
       __syncthreads();
       // the tile's keys and values, 16 bytes a load: four threads share a key (its page is looked
       // up once per thread and tile) and take its pieces in turn, LOADS pieces of each kind in
@@ -135,7 +139,7 @@ attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ pages, T* _
       {
         const int n = tid >> 2, key = n0 + n;
         const T* kp = nullptr;
-        if (key < s_hi && key >= key_lo_tile)
+        if (key < s_hi && ls_sees(key, key_lo_tile, keep_first))
           kp = page_ptr<T>(pages, table_row, key, 0, kvh, nkv, page_size, d, num_pages, err);
         const int64_t to_v = (int64_t)nkv * page_size * d;
         for (int ch0 = tid & 3; ch0 < pieces; ch0 += 4 * LOADS) {
@@ -191,7 +195,7 @@ attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ pages, T* _
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int key = n0 + sub + 8 * j;
-          const bool keep = key < s_hi && key <= qpos && key >= row_lo;
+          const bool keep = key < s_hi && key <= qpos && ls_sees(key, row_lo, keep_first);
           s[j] = !keep ? -CUDART_INF_F
                  : log_rates != nullptr ? ls_capped(dot[j] * scale, softcap) - slope * log1pf(log_rate * (float)(qpos - key))
                  : slopes != nullptr ? fmaf(slope, (float)(key - qpos), ls_capped(dot[j] * scale, softcap)) : ls_capped(dot[j] * scale, softcap);
@@ -317,7 +321,7 @@ attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ pages,
                         float* __restrict__ part_acc, float* __restrict__ part_ml,
                         const int* __restrict__ work, const int* __restrict__ block_table,
                         int table_stride, int nq, int nkv, int d, int page_size, int num_pages,
-                        int window, float scale, float softcap, const float* __restrict__ slopes,
+                        int window, int keep_first, float scale, float softcap, const float* __restrict__ slopes,
                         const float* __restrict__ log_rates, int slot_limit, int* err) {
   ls_dependency_sync();
   extern __shared__ __align__(16) unsigned char dsm[];
@@ -364,15 +368,16 @@ attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ pages,
 
   const int cpr = d / VEC;                   // 16-byte chunks per row
   int t_first = s_lo;
-  if (row_lo > s_lo) t_first = s_lo + ((row_lo - s_lo) / DEC_TILE) * DEC_TILE;
+  if (row_lo > s_lo && s_lo >= keep_first) t_first = s_lo + ((row_lo - s_lo) / DEC_TILE) * DEC_TILE;
 
   for (int n0 = t_first; n0 < s_hi; n0 += DEC_TILE) {
+    if (n0 >= keep_first && n0 + DEC_TILE <= row_lo) continue;
     __syncthreads();
     for (int i = tid; i < DEC_TILE * cpr; i += 128) {
       const int n = i / cpr, c = i - n * cpr;
       const int key = n0 + n;
       uint4 kv = make_uint4(0, 0, 0, 0), vv = make_uint4(0, 0, 0, 0);
-      if (key < s_hi && key >= row_lo) {
+      if (key < s_hi && ls_sees(key, row_lo, keep_first)) {
         const T* kp = page_ptr<T>(pages, table_row, key, 0, kvh, nkv, page_size, d, num_pages, err);
         if (kp != nullptr) {
           kv = *reinterpret_cast<const uint4*>(kp + c * VEC);
@@ -396,7 +401,7 @@ attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ pages,
 #pragma unroll
         for (int x = 0; x < VEC; ++x) dot = fmaf(qr[c + x], ls_to_float<T>(e[x]), dot);
       }
-      const bool keep = key < s_hi && key >= row_lo;
+      const bool keep = key < s_hi && ls_sees(key, row_lo, keep_first);
       Ss[u] = !keep ? -CUDART_INF_F
               : log_rates != nullptr ? ls_capped(dot * scale, softcap) - slopes[kvh * group + g] * log1pf(log_rates[kvh * group + g] * (float)(pos - key))
               : slopes != nullptr ? fmaf(slopes[kvh * group + g], (float)(key - pos), ls_capped(dot * scale, softcap)) : ls_capped(dot * scale, softcap);
@@ -501,10 +506,11 @@ LS_API int ls_attention_split_size() { return LS_SPLIT; }
 LS_API int ls_attention_tile(const void* q, const void* pages, void* out, float* part_acc,
                              float* part_ml, int dtype, const int* work, int n_work,
                              const int* block_table, int table_stride, int nq, int nkv, int d,
-                             int page_size, int num_pages, int window, float scale, float softcap,
+                             int page_size, int num_pages, int window, int keep_first, float scale, float softcap,
                              const float* slopes, const float* log_rates, const float* sinks, int* err,
                              cudaStream_t stream) {
   if (n_work <= 0) return 0;
+  if (keep_first < 0) return LS_E_SIZE;
   if (log_rates != nullptr && slopes == nullptr) return LS_E_SIZE;
   if (!shape_ok(nq, nkv, d, page_size, LS_SPLIT)) return LS_E_SIZE;
   if (nq > 65535) return LS_E_SIZE;
@@ -526,7 +532,7 @@ LS_API int ls_attention_tile(const void* q, const void* pages, void* out, float*
     if (smem > set_f32) set_f32 = smem;
     LS_COUNT(LS_K_ATTENTION_TILE), ls_launch(attention_tile_kernel<float>, grid, 128, smem, stream, 
         (const float*)q, (const float*)pages, (float*)out, part_acc, part_ml, work, block_table,
-        table_stride, nq, nkv, d, page_size, num_pages, window, scale, softcap, slopes, log_rates, sinks, hb, err);
+        table_stride, nq, nkv, d, page_size, num_pages, window, keep_first, scale, softcap, slopes, log_rates, sinks, hb, err);
   } else if (dtype == LS_BF16) {
     e = smem <= set_bf16 ? cudaSuccess
                          : cudaFuncSetAttribute(attention_tile_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -534,7 +540,7 @@ LS_API int ls_attention_tile(const void* q, const void* pages, void* out, float*
     if (smem > set_bf16) set_bf16 = smem;
     LS_COUNT(LS_K_ATTENTION_TILE), ls_launch(attention_tile_kernel<__nv_bfloat16>, grid, 128, smem, stream, 
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)pages, (__nv_bfloat16*)out, part_acc,
-        part_ml, work, block_table, table_stride, nq, nkv, d, page_size, num_pages, window, scale,
+        part_ml, work, block_table, table_stride, nq, nkv, d, page_size, num_pages, window, keep_first, scale,
         softcap, slopes, log_rates, sinks, hb, err);
   } else {
     return LS_E_DTYPE;
@@ -548,7 +554,7 @@ namespace {
 int launch_attention_decode(const void* q, const void* pages, float* part_acc, float* part_ml,
                             int dtype, const int* work, int n_work, const int* block_table,
                             int table_stride, int nq, int nkv, int d, int page_size,
-                            int num_pages, int window, float scale, float softcap, const float* slopes,
+                            int num_pages, int window, int keep_first, float scale, float softcap, const float* slopes,
                             const float* log_rates, int slot_limit, int* err, cudaStream_t stream) {
   if (n_work <= 0) return 0;
   if (log_rates != nullptr && slopes == nullptr) return LS_E_SIZE;
@@ -566,7 +572,7 @@ int launch_attention_decode(const void* q, const void* pages, float* part_acc, f
     if (smem > set_f32) set_f32 = smem;
     LS_COUNT(LS_K_ATTENTION_DECODE), ls_launch(attention_decode_kernel<float>, grid, 128, smem, stream, 
         (const float*)q, (const float*)pages, part_acc, part_ml, work, block_table, table_stride,
-        nq, nkv, d, page_size, num_pages, window, scale, softcap, slopes, log_rates, slot_limit, err);
+        nq, nkv, d, page_size, num_pages, window, keep_first, scale, softcap, slopes, log_rates, slot_limit, err);
   } else if (dtype == LS_BF16) {
     const size_t smem = decode_smem_bytes(d, group, 2);
     e = smem <= set_bf16 ? cudaSuccess
@@ -575,7 +581,7 @@ int launch_attention_decode(const void* q, const void* pages, float* part_acc, f
     if (smem > set_bf16) set_bf16 = smem;
     LS_COUNT(LS_K_ATTENTION_DECODE), ls_launch(attention_decode_kernel<__nv_bfloat16>, grid, 128, smem, stream, 
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)pages, part_acc, part_ml, work,
-        block_table, table_stride, nq, nkv, d, page_size, num_pages, window, scale, softcap, slopes, log_rates, slot_limit, err);
+        block_table, table_stride, nq, nkv, d, page_size, num_pages, window, keep_first, scale, softcap, slopes, log_rates, slot_limit, err);
   } else {
     return LS_E_DTYPE;
   }
@@ -605,10 +611,11 @@ int launch_attention_combine(const float* part_acc, const float* part_ml, void* 
 LS_API int ls_attention_decode(const void* q, const void* pages, float* part_acc, float* part_ml,
                                int dtype, const int* work, int n_work, const int* block_table,
                                int table_stride, int nq, int nkv, int d, int page_size,
-                               int num_pages, int window, float scale, float softcap, const float* slopes,
+                               int num_pages, int window, int keep_first, float scale, float softcap, const float* slopes,
                                const float* log_rates, int* err, cudaStream_t stream) {
+  if (keep_first < 0) return LS_E_SIZE;
   return launch_attention_decode(q, pages, part_acc, part_ml, dtype, work, n_work, block_table, table_stride, nq,
-                                 nkv, d, page_size, num_pages, window, scale, softcap, slopes, log_rates, 0, err, stream);
+                                 nkv, d, page_size, num_pages, window, keep_first, scale, softcap, slopes, log_rates, 0, err, stream);
 }
 
 LS_API int ls_attention_combine(const float* part_acc, const float* part_ml, void* out, int dtype,
@@ -671,7 +678,7 @@ LS_API int ls_attention_decode_noalloc(const void* q, const void* pages, void* o
   // in the error word (LS_DEV_ROW_RANGE) and skipped, it cannot write outside the array
   const int status = launch_attention_decode(q, pages, part_acc, part_ml, dtype, work, n_work,
                                              block_table, table_stride, nq, nkv, d, page_size,
-                                             num_pages, window, scale, 0.f, nullptr, nullptr, n_slots, err, stream);
+                                             num_pages, window, 0, scale, 0.f, nullptr, nullptr, n_slots, err, stream);
   if (status != 0) return status;
   return launch_attention_combine(part_acc, part_ml, out, dtype, combine, n_combine, nq, d, n_slots, nullptr, err, stream);
 }

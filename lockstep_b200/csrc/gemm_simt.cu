@@ -13,6 +13,7 @@
 //   1 residual     C[m, n] += acc                       (C float32, in place)
 //   2 silu-mul     C[m, n]  = silu(acc_gate) * acc_up   (W holds gate rows [0, N)
 //                                                        and up rows [N, 2N))
+//   4 gelu         C[m, n]  = gelu_tanh(acc)
 #include "common.cuh"
 
 namespace {
@@ -85,6 +86,8 @@ gemm_nt_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TC* __restric
         *c = ls_from_float<TC>(acc[i][j]);
       } else if (EPI == 1) {
         *c = ls_from_float<TC>(ls_to_float<TC>(*c) + acc[i][j]);
+      } else if (EPI == 4) {
+        *c = ls_from_float<TC>(ls_gelu_tanh(acc[i][j]));
       } else {
         const float g = acc[i][j];
         *c = ls_from_float<TC>(g / (1.0f + expf(-g)) * acu[i][j]);
@@ -211,6 +214,8 @@ gemm_nt_skinny_kernel(const float* __restrict__ A, const float* __restrict__ W, 
         *c = ls_from_float<TC>(acc[i]);
       } else if (EPI == 1) {
         *c = ls_from_float<TC>(ls_to_float<TC>(*c) + acc[i]);
+      } else if (EPI == 4) {
+        *c = ls_from_float<TC>(ls_gelu_tanh(acc[i]));
       } else {
         const float g = acc[i];
         *c = ls_from_float<TC>(g / (1.0f + expf(-g)) * acu[i]);
@@ -369,7 +374,7 @@ gemm_nt_large_kernel(const float* __restrict__ A, const float* __restrict__ W, f
 #pragma unroll
       for (int j = 0; j < WC; ++j) {
         const int n = n0 + (j < 4 ? tx * 4 + j : 64 + tx * 4 + j - 4);
-        if (n < N) crow[n] = EPI == 1 ? crow[n] + acc[i][j] : acc[i][j];
+        if (n < N) crow[n] = EPI == 1 ? crow[n] + acc[i][j] : EPI == 4 ? ls_gelu_tanh(acc[i][j]) : acc[i][j];
       }
     }
   }
@@ -423,6 +428,9 @@ int launch(const void* A, const void* W, void* C, int M, int N, int K, int64_t l
     case 2:
       LS_COUNT(LS_K_GEMM_SIMT), ls_launch(gemm_nt_kernel<TA, TW, TC, 2>, grid, 256, 0, stream, (const TA*)A, (const TW*)W, (TC*)C, M, N, K, lda, ldw, ldc);
       break;
+    case 4:
+      LS_COUNT(LS_K_GEMM_SIMT), ls_launch(gemm_nt_kernel<TA, TW, TC, 4>, grid, 256, 0, stream, (const TA*)A, (const TW*)W, (TC*)C, M, N, K, lda, ldw, ldc);
+      break;
     default:
       return LS_E_SIZE;
   }
@@ -446,6 +454,7 @@ LS_API int ls_gemm_nt_simt(const void* A, const void* W, void* C, int a_dtype, i
     if (epilogue == 0) return launch_skinny<0>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     if (epilogue == 1) return launch_skinny<1>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     if (epilogue == 2) return launch_skinny<2>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
+    if (epilogue == 4) return launch_skinny<4>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     return LS_E_SIZE;
   }
   // float32 rows that can be fetched 16 bytes at a time, more than a few of them
@@ -456,6 +465,7 @@ LS_API int ls_gemm_nt_simt(const void* A, const void* W, void* C, int a_dtype, i
     if (epilogue == 0) return launch_large<0>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     if (epilogue == 1) return launch_large<1>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     if (epilogue == 2) return launch_large<2>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
+    if (epilogue == 4) return launch_large<4>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     return LS_E_SIZE;
   }
   if (a_dtype == LS_F32 && c_dtype == LS_F32)

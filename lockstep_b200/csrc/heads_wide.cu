@@ -4,14 +4,16 @@
 //   - key heads of size d and value heads of size dv that need not be equal;
 //   - a layer that projects queries only (it reads another layer's keys and values);
 //   - biases of the three projections, added here (in float32) rather than in the product;
-//   - a query temperature: the query of position p times 1 + coef ln(floor((p + 1) / every) + 1).
+//   - a query temperature: the query of position p times 1 + coef ln(floor((p + 1) / every) + 1);
+//   - rotation of neighbouring pairs (2i, 2i + 1) instead of (i, i + rot_dim / 2);
+//   - values mixed with another projection's values of the same token: v <- (1 - mix) v + mix other.
 // Queries go to q_out [tokens, nq * D], keys and values into the cache pages
 // [num_pages, 2, nkv, page_size, D]; D >= max(d, dv) is the one head size the attention
 // kernels then work with, and the elements past d (dv) are written as zeros: a zero in a
 // query or key adds nothing to a score, a zero value column gives a zero output column.
 // One block per token.  Sums of squares are taken in float32 in a fixed order (a thread's
 // elements ascending, lanes by xor-tree, warps ascending), so a token's bits do not depend
-// on the batch.  Rotation: the halves layout on the first rot_dim elements of each head,
+// on the batch.  Rotation: halves or neighbouring pairs of the first rot_dim elements of each head,
 // products and sums rounded one by one as in rope.cuh.
 #include "common.cuh"
 
@@ -39,6 +41,10 @@ struct WideArgs {
   int bias_bf16;
   float temp_coef;          // query temperature (0: none)
   int temp_every;
+  int interleaved;
+  const void* v_other;      // null, or [tokens, v_other_ld]: values to mix into this layer's
+  int64_t v_other_ld;
+  const float* v_mix;       // one number
 };
 
 __device__ __forceinline__ float gain_at(const void* g, int bf16, int i) {
@@ -96,7 +102,12 @@ __device__ void finish_heads(const WideArgs& a, const T* src, int col0, int head
         }
         return v;
       };
-      if (i < a.rot_dim) {
+      if (i < a.rot_dim && a.interleaved) {
+        const int r = i >> 1;
+        const float lo = normed(2 * r), hi = normed(2 * r + 1);
+        out = (i & 1) == 0 ? __fsub_rn(__fmul_rn(lo, cs[r]), __fmul_rn(hi, sn[r]))
+                           : __fadd_rn(__fmul_rn(hi, cs[r]), __fmul_rn(lo, sn[r]));
+      } else if (i < a.rot_dim) {
         if (i < half) {
           const float lo = normed(i), hi = normed(i + half);
           out = __fsub_rn(__fmul_rn(lo, cs[i]), __fmul_rn(hi, sn[i]));
@@ -160,10 +171,16 @@ __global__ void __launch_bounds__(THREADS) qkv_finish_kernel(WideArgs a, int* er
   finish_heads<T>(a, k_src, a.nq * a.d, a.nkv, a.k_gain, k_rstd, cs, sn, head_rstd, 1.0f, [&](int h, int i, float v) {
     pages[((((int64_t)page * 2 + 0) * a.nkv + h) * a.page_size + in_page) * a.D + i] = ls_from_float<T>(v);
   });
+  const T* other = a.v_other != nullptr ? reinterpret_cast<const T*>(a.v_other) + (int64_t)t * a.v_other_ld : nullptr;
+  const float mix = other != nullptr ? *a.v_mix : 0.f;
   for (int e = threadIdx.x; e < a.nkv * a.D; e += THREADS) {
     const int h = e / a.D, i = e - h * a.D;
-    pages[((((int64_t)page * 2 + 1) * a.nkv + h) * a.page_size + in_page) * a.D + i] =
-        i < a.dv ? ls_from_float<T>(biased_at<T>(a, v_src, (a.nq + a.nkv) * a.d, h * a.dv + i)) : ls_from_float<T>(0.f);
+    float v = 0.f;
+    if (i < a.dv) {
+      v = biased_at<T>(a, v_src, (a.nq + a.nkv) * a.d, h * a.dv + i);
+      if (other != nullptr) v = __fadd_rn(__fmul_rn(1.0f - mix, v), __fmul_rn(mix, ls_to_float<T>(other[h * a.dv + i])));
+    }
+    pages[((((int64_t)page * 2 + 1) * a.nkv + h) * a.page_size + in_page) * a.D + i] = ls_from_float<T>(v);
   }
 }
 
@@ -174,8 +191,8 @@ LS_API int ls_qkv_finish(const void* qkv, int64_t ld, void* q_out, void* pages, 
                          const int* positions, const int* token_req, const int* block_table, int table_stride,
                          int tokens, int nq, int nkv, int d, int dv, int D, int rot_dim, int page_size,
                          int num_pages, int max_positions, float eps, int scope, int has_kv, int write_cache,
-                         const void* bias, int bias_dtype, float temp_coef, int temp_every,
-                         int* err, cudaStream_t stream) {
+                         const void* bias, int bias_dtype, float temp_coef, int temp_every, int interleaved,
+                         const void* v_other, int64_t v_other_ld, const float* v_mix, int* err, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || D < d || D < dv || scope < 0 || scope > 2) return LS_E_SIZE;
   if (rot_dim < 0 || rot_dim > d || (rot_dim & 1)) return LS_E_SIZE;
@@ -184,7 +201,9 @@ LS_API int ls_qkv_finish(const void* qkv, int64_t ld, void* q_out, void* pages, 
   if (write_cache && (pages == nullptr || page_size <= 0)) return LS_E_SIZE;
   if (temp_coef != 0.f && temp_every <= 0) return LS_E_SIZE;
   if (bias != nullptr && bias_dtype != LS_F32 && bias_dtype != LS_BF16) return LS_E_DTYPE;
+  if (v_other != nullptr && (v_mix == nullptr || !has_kv || v_other_ld < (int64_t)nkv * dv)) return LS_E_SIZE;
   WideArgs a;
+  a.interleaved = interleaved; a.v_other = v_other; a.v_other_ld = v_other_ld; a.v_mix = v_mix;
   a.bias = bias; a.bias_bf16 = bias_dtype == LS_BF16 ? 1 : 0; a.temp_coef = temp_coef; a.temp_every = temp_every > 0 ? temp_every : 1;
   a.qkv = qkv; a.q_out = q_out; a.pages = pages; a.q_gain = q_gain; a.k_gain = k_gain;
   a.cos_table = cos_table; a.sin_table = sin_table; a.positions = positions; a.token_req = token_req;

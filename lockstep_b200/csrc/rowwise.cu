@@ -7,7 +7,8 @@
 //   - an embedding with a factor on the token's row and a second table indexed by a hash of the
 //     token and the one before it, whose last row serves a sequence's first token;
 //   - float32 rows written into some columns of a wider row of the engine's type; logits times a
-//     factor, then capped with tanh.
+//     factor, then capped with tanh;
+//   - the gate of a token's own embedding in a layer: gelu(z) times some columns of the token's row of a table.
 // All reductions run in float32 in an order fixed by the row's own width (a thread's elements
 // ascending, the lanes by an xor tree, the warps ascending), so a row's result does not depend on the batch.
 #include "common.cuh"
@@ -187,6 +188,26 @@ __global__ void scale_cap_kernel(float* __restrict__ x, int64_t count, float fac
   }
 }
 
+// out[t, c] = gelu_tanh(z[t, c]) table[ids[t], at + c]
+template <typename T>
+__global__ void side_gate_kernel(const float* __restrict__ z, const int* __restrict__ ids, const T* __restrict__ table,
+                                 int64_t table_ld, int at, int vocab, T* __restrict__ out, int64_t tokens, int dim, int* err) {
+  ls_dependency_sync();
+  const int64_t n = tokens * dim;
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = i / dim;
+    const int c = (int)(i - t * dim);
+    const int id = ids[t];
+    float v = 0.f;
+    if (id < 0 || id >= vocab) {
+      if (c == 0) ls_record_fault(err, LS_DEV_TOKEN_RANGE, (int)t);
+    } else {
+      v = ls_gelu_tanh(z[i]) * ls_to_float<T>(table[id * table_ld + at + c]);
+    }
+    out[i] = ls_from_float<T>(v);
+  }
+}
+
 inline int blocks_for(int64_t n) { return (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16); }
 
 }  // namespace
@@ -256,6 +277,21 @@ LS_API int ls_rows_cast(const float* src, void* dst, int dst_dtype, long long ro
   LS_COUNT(LS_K_ROWS_CAST);
   if (dst_dtype == LS_F32) ls_launch(rows_cast_kernel<float>, blocks_for(rows * width), 256, 0, stream, src, (float*)dst, (int64_t)rows, width, (int64_t)ld);
   else if (dst_dtype == LS_BF16) ls_launch(rows_cast_kernel<__nv_bfloat16>, blocks_for(rows * width), 256, 0, stream, src, (__nv_bfloat16*)dst, (int64_t)rows, width, (int64_t)ld);
+  else return LS_E_DTYPE;
+  return ls_launch_status();
+}
+
+LS_API int ls_side_gate(const float* z, const int* ids, const void* table, long long table_ld, int at, int vocab, void* out,
+                        int dtype, long long tokens, int dim, int* err, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (dim <= 0 || at < 0 || at + dim > table_ld || vocab <= 0) return LS_E_SIZE;
+  LS_COUNT(LS_K_SIDE_GATE);
+  if (dtype == LS_F32)
+    ls_launch(side_gate_kernel<float>, blocks_for(tokens * dim), 256, 0, stream, z, ids, (const float*)table, (int64_t)table_ld,
+              at, vocab, (float*)out, (int64_t)tokens, dim, err);
+  else if (dtype == LS_BF16)
+    ls_launch(side_gate_kernel<__nv_bfloat16>, blocks_for(tokens * dim), 256, 0, stream, z, ids, (const __nv_bfloat16*)table,
+              (int64_t)table_ld, at, vocab, (__nv_bfloat16*)out, (int64_t)tokens, dim, err);
   else return LS_E_DTYPE;
   return ls_launch_status();
 }

@@ -171,10 +171,6 @@ struct ScanArgs {
   int width, taps;
 };
 
-__device__ __forceinline__ float gelu_tanh_f(float z) {
-  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-}
-
 template <typename T>
 __global__ void __launch_bounds__(128) unit_scan_kernel(ScanArgs s) {
   ls_dependency_sync();
@@ -202,7 +198,7 @@ __global__ void __launch_bounds__(128) unit_scan_kernel(ScanArgs s) {
     for (int k = 0; k < AHEAD; ++k) {
       if (i0 + k >= n) break;
       S = fmaf(a[k], S, b[k]);
-      out[(int64_t)(t0 + i0 + k) * s.width + c] = ls_from_float<T>(S * gelu_tanh_f(y[k] + yb));
+      out[(int64_t)(t0 + i0 + k) * s.width + c] = ls_from_float<T>(S * ls_gelu_tanh(y[k] + yb));
     }
   }
   state[c] = S;

@@ -47,19 +47,34 @@ def first_key(pos, window: int):
     return pos * 0
 
 
-def plan_attention(portions, window: int, split_size: int, tile_tokens: int = TILE_TOKENS):
-    """portions: (slot, token offset, start position, length) per entry.
+def mask_parts(mask) -> tuple[int, int]:
+    """(window, keep_first) of a mask: a window as ``first_key`` takes it, or a pair (window, keep_first) whose first
+    ``keep_first`` positions of the sequence stay visible wherever the window is."""
+    return (int(mask[0]), int(mask[1])) if isinstance(mask, tuple) else (int(mask), 0)
+
+
+def kept_splits(pos, mask, split_size: int):
+    """How many leading splits hold first keys that a query at ``pos`` (a number or an array) reads although they
+    lie before the splits of its window."""
+    window, keep = mask_parts(mask)
+    return np.minimum(-(-keep // split_size), first_key(pos, window) // split_size) if keep else pos * 0
+
+
+def plan_attention(portions, mask, split_size: int, tile_tokens: int = TILE_TOKENS):
+    """portions: (slot, token offset, start position, length) per entry.  ``mask``: see ``mask_parts``.
     Returns numpy arrays (tile_work [n,8], split_work [n,8], combine [n,4]) and
     the number of scratch slots.  Tiles hold up to ``tile_tokens`` tokens and are
     listed longest context first, so that the heaviest start first."""
     tile, split, combine = [], [], []
     n_slots = 0
+    window, _ = mask_parts(mask)
     for slot, off, start, length in portions:
         if length == 1:
             lo = first_key(start, window)
             s_lo, s_hi = lo // split_size, start // split_size
-            combine.append((off, n_slots, 1, s_hi - s_lo + 1))
-            for s in range(s_lo, s_hi + 1):
+            lead = int(kept_splits(start, mask, split_size))
+            combine.append((off, n_slots, 1, lead + s_hi - s_lo + 1))
+            for s in [*range(lead), *range(s_lo, s_hi + 1)]:
                 split.append((slot, off, 1, start, s, s + 1, n_slots, 0))
                 n_slots += 1
         else:
@@ -68,7 +83,7 @@ def plan_attention(portions, window: int, split_size: int, tile_tokens: int = TI
                 pos0 = start + i
                 lo = first_key(pos0, window)
                 tile.append((slot, off + i, ntok, pos0, lo // split_size,
-                             (pos0 + ntok - 1) // split_size + 1, -1, 0))
+                             (pos0 + ntok - 1) // split_size + 1, -1, int(kept_splits(pos0, mask, split_size))))
     tile.sort(key=lambda item: -(item[3] + item[2]))
     as_np = lambda rows, w: np.asarray(rows, dtype=np.int32).reshape(-1, w)
     return as_np(tile, 8), as_np(split, 8), as_np(combine, 4), n_slots
@@ -105,10 +120,10 @@ class StepContext:
         self.positions = dev[t:2 * t]
         self.token_slot = dev[2 * t:3 * t]
         self.wanted_rows = dev[3 * t:3 * t + self.n_wanted]
-        self._plans: dict[tuple[int, int], AttentionPlan] = {}
+        self._plans: dict[tuple, AttentionPlan] = {}
 
-    def attention_plan(self, window: int, tile_tokens: int = TILE_TOKENS) -> AttentionPlan:
-        """Work lists for attention with ``window`` (0: all keys): portions of two or
+    def attention_plan(self, window, tile_tokens: int = TILE_TOKENS) -> AttentionPlan:
+        """Work lists for attention with the mask ``window`` (0: all keys; see ``mask_parts``): portions of two or
         more tokens cut into tiles of ``tile_tokens``, single tokens into one item
         per split plus a combine item."""
         plan = self._plans.get((window, tile_tokens))

@@ -36,7 +36,7 @@ from collections import OrderedDict
 import numpy as np
 import torch
 
-from .batch import AttentionPlan, first_key, plan_attention
+from .batch import AttentionPlan, first_key, kept_splits, mask_parts, plan_attention
 
 CAPACITY_STEP = 32      # the attention work list of a recorded step holds a multiple of this many items
 MAX_GRAPHS = 24         # recorded steps kept; the least recently used one goes first
@@ -51,7 +51,7 @@ def padded_batch(n: int) -> int:
 class StaticStepContext:
     """What parts see of a recorded decode step: views into the graph's buffer."""
 
-    def __init__(self, batch: int, capacity: int, windows: list[int], device, err, split_size: int,
+    def __init__(self, batch: int, capacity: int, windows: list, device, err, split_size: int,
                  pad_slot: int = 0):
         self.batch, self.capacity, self.windows = batch, capacity, list(windows)
         self.pad_slot = pad_slot
@@ -65,8 +65,8 @@ class StaticStepContext:
         b = batch
         self.token_ids, self.positions = self.dev[0:b], self.dev[b:2 * b]
         self.token_slot, self.wanted_rows = self.dev[2 * b:3 * b], self.dev[3 * b:4 * b]
-        self._plans: dict[int, AttentionPlan] = {}
-        self._offsets: dict[int, int] = {}
+        self._plans: dict[object, AttentionPlan] = {}
+        self._offsets: dict[object, int] = {}
         off = 4 * b
         for w in self.windows:
             self._offsets[w] = off
@@ -83,7 +83,7 @@ class StaticStepContext:
         self.copied = torch.cuda.Event()
         self._pending = False
 
-    def attention_plan(self, window: int, tile_tokens: int = 0) -> AttentionPlan:
+    def attention_plan(self, window, tile_tokens: int = 0) -> AttentionPlan:
         try:
             return self._plans[window]
         except KeyError:
@@ -108,17 +108,20 @@ class StaticStepContext:
         h[2 * b:3 * b] = slot
         h[3 * b:4 * b] = self._arange
         for w in self.windows:
-            # one item per (entry, split): splits lo // S .. start // S of each entry, in entry order
-            lo = first_key(start, w)
+            # one item per (entry, split), in entry order: the leading splits of kept first keys, then lo // S .. start // S
+            lo = first_key(start, mask_parts(w)[0])
+            lead = kept_splits(start, w, self.split_size)
             first, last = lo // self.split_size, start // self.split_size
-            count = last - first + 1
+            count = lead + last - first + 1
             count[n:] = 0                  # padding rows attend to nothing: no items, an empty combine
             total = int(count.sum())
             if total > self.capacity:
                 raise ValueError("the attention work list outgrew the capacity this graph was recorded for")
             base = np.cumsum(count) - count                       # first scratch slot of each entry
             owner = np.repeat(np.arange(b), count)
-            split = np.arange(total) - np.repeat(base, count) + np.repeat(first, count)
+            rank = np.arange(total) - np.repeat(base, count)      # place among the entry's own splits
+            ahead = np.repeat(lead, count)
+            split = np.where(rank < ahead, rank, rank - ahead + np.repeat(first, count))
             off = self._offsets[w]
             items = h[off:off + self.capacity * 8].reshape(self.capacity, 8)
             items[:total, 0] = slot[owner]
@@ -156,10 +159,10 @@ class StaticMixedContext:
     logits are dropped, and with null items, which the kernels skip)."""
 
     def __init__(self, tokens: int, wanted_cap: int, split_cap: int, max_entries: int,
-                 plan_keys: list[tuple[int, int]], device, err, split_size: int):
+                 plan_keys: list[tuple], device, err, split_size: int):
         self.num_tokens, self.n_wanted = tokens, wanted_cap
         self.split_cap, self.max_entries = split_cap, max_entries
-        self.plan_keys = sorted(plan_keys)
+        self.plan_keys = sorted(plan_keys, key=lambda key: (mask_parts(key[0]), key[1]))
         self.device, self.err, self.split_size = device, err, split_size
         t = tokens
         # (a few items more than the tokens make in one portion: a launcher that chooses a kernel
@@ -193,7 +196,7 @@ class StaticMixedContext:
         self._pending = False
         self.wanted = 0
 
-    def attention_plan(self, window: int, tile_tokens: int = 16) -> AttentionPlan:
+    def attention_plan(self, window, tile_tokens: int = 16) -> AttentionPlan:
         try:
             return self._plans[(window, tile_tokens)]
         except KeyError:
@@ -236,14 +239,14 @@ class StaticMixedContext:
         self._pending = True
 
 
-def split_items(entries, windows: list[int], split_size: int) -> int:
+def split_items(entries, windows: list, split_size: int) -> int:
     """The longest attention work list of a decode step over ``entries``."""
     worst = 0
     for w in windows:
         n = 0
         for e in entries:
-            lo = first_key(e.start, w)
-            n += e.start // split_size - lo // split_size + 1
+            lo = first_key(e.start, mask_parts(w)[0])
+            n += int(kept_splits(e.start, w, split_size)) + e.start // split_size - lo // split_size + 1
         worst = max(worst, n)
     return worst
 
@@ -251,7 +254,7 @@ def split_items(entries, windows: list[int], split_size: int) -> int:
 class DecodeGraphs:
     def __init__(self, runner, round_to: int = CAPACITY_STEP, max_graphs: int = MAX_GRAPHS):
         self.runner, self.round_to, self.max_graphs = runner, round_to, max(1, int(max_graphs))
-        self.windows = sorted(set().union(*(b.attention_windows() for b in runner.model.blocks)) or {0})
+        self.windows = sorted(set().union(*(b.attention_windows() for b in runner.model.blocks)) or {0}, key=mask_parts)
         self.graphs: OrderedDict[tuple[int, int], tuple] = OrderedDict()
         self.pool = None
         self.replays = 0

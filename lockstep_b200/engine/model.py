@@ -19,6 +19,8 @@ from ..parts import Runtime, WeightSpec, build_part
 class Model:
     def __init__(self, spec: ModelSpec, runtime: Runtime):
         self.spec, self.rt = spec, runtime
+        self.shared = {name: build_part("table", part, runtime) for name, part in spec.shared.items()}
+        runtime.shared.update(self.shared)
         self.embedding = build_part("embedding", spec.embedding, runtime)
         self.blocks = [build_part("block", layer.block, runtime, layer_spec=layer) for layer in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm, runtime)
@@ -40,6 +42,8 @@ class Model:
         yield n["head"], self.head
         if self.injection is not None:
             yield n["injection"], self.injection
+        for name, part in self.shared.items():
+            yield n[name], part
 
     def weight_specs(self) -> dict[str, WeightSpec]:
         out: dict[str, WeightSpec] = {}

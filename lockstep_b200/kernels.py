@@ -19,7 +19,7 @@ from .csrc import build as _build
 F32, BF16 = 0, 1
 _DTYPE_CODE = {torch.float32: F32, torch.bfloat16: BF16}
 
-EPILOGUE_STORE, EPILOGUE_RESIDUAL, EPILOGUE_SILU_MUL = 0, 1, 2
+EPILOGUE_STORE, EPILOGUE_RESIDUAL, EPILOGUE_SILU_MUL, EPILOGUE_GELU = 0, 1, 2, 4
 FEW_TOKENS = 32      # up to here a product runs in the few-token kernel, which can also finish q/k/v heads
 
 _REFUSALS = {
@@ -60,6 +60,8 @@ _SIGNATURES = {
                           c_int, c_int, ctypes.c_longlong, ctypes.c_longlong, c_float, c_void_p, c_void_p],
         "ls_rows_cast": [c_void_p, c_void_p, c_int, ctypes.c_longlong, c_int, ctypes.c_longlong, c_void_p],
         "ls_scale_cap": [c_void_p, ctypes.c_longlong, c_float, c_float, c_void_p],
+        "ls_side_gate": [c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int, c_void_p, c_int, ctypes.c_longlong,
+                         c_int, c_void_p, c_void_p],
         "ls_row_bias": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "ls_weighted_sum": [c_void_p, c_void_p, ctypes.c_longlong, c_int, ctypes.POINTER(c_float), c_void_p, c_int,
                             c_void_p],
@@ -72,10 +74,10 @@ _SIGNATURES = {
                             c_int64, c_int64, c_int64, c_int, c_void_p],
         "ls_attention_split_size": [],
         "ls_attention_tile": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
-                              c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                              c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                               c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
         "ls_attention_decode": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
-                                c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
+                                c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
                                 c_void_p, c_void_p, c_void_p, c_void_p],
         "ls_attention_combine": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
                                  c_void_p, c_void_p],
@@ -89,10 +91,12 @@ _SIGNATURES["tc"] = {
     "ls_gemm_tc_token_tile": [c_int, c_int, c_int, c_int],
     "ls_gemm_tc_k_shares": [c_int, c_int],
     "ls_attention_decode_mma": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
-                                c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
+                                c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p,
+                                c_void_p, c_void_p],
     "ls_attention_prefill_tc_tile_tokens": [],
     "ls_attention_prefill_tc": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                                c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p],
+                                c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
+                                c_void_p],
     "ls_gemm_nt_tc_qkv_heads": [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p,
                                 c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                 c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -106,7 +110,8 @@ _SIGNATURES["tc"] = {
 _SIGNATURES["seq"] = {
     "ls_qkv_finish": [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                       c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                      c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p],
+                      c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_int, c_float, c_int, c_int, c_void_p,
+                      c_int64, c_void_p, c_void_p, c_void_p],
     "ls_latent_finish": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                          c_int, c_float, c_void_p, c_void_p, c_void_p],
@@ -115,13 +120,13 @@ _SIGNATURES["seq"] = {
     "ls_sigmoid_power_decay": [c_void_p, c_void_p, ctypes.c_longlong, c_int, c_float, c_void_p],
     "ls_find_portions": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p],
     "ls_delta_prep": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p,
-                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
+                      c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
     "ls_double_exp_decay": [c_void_p, c_void_p, ctypes.c_longlong, c_int, c_void_p],
     "ls_shift_mix": [c_void_p, c_int, c_void_p, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_int, c_int, c_int,
                      c_void_p],
     "ls_state_rule": [c_int, c_int, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
                       c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
-                      c_int64, c_float, c_int64, c_void_p],
+                      c_int64, c_float, c_int64, c_void_p, c_float, c_void_p],
     "ls_unit_gates": [c_void_p, ctypes.c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong,
                       c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                       c_int, c_float, c_void_p],
@@ -130,7 +135,7 @@ _SIGNATURES["seq"] = {
     "ls_rotate_rows": [c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                        c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     "ls_head_rms_gate": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                         c_float, c_int64, c_void_p],
+                         c_float, c_int64, c_int, c_void_p],
     "ls_tanh_rows": [c_void_p, c_int, ctypes.c_longlong, c_void_p],
     "ls_experts_tile_rows": [],
     "ls_experts_route": [c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
@@ -495,6 +500,17 @@ def scale_cap(x, factor: float, cap: float) -> None:
     _check(library().ls_scale_cap(_dev(x, "x", torch.float32), x.numel(), float(factor), float(cap), _stream()), "scale_cap")
 
 
+def side_gate(z, ids, table, at: int, out, err) -> None:
+    """out[t, c] = gelu(z[t, c]) table[ids[t], at + c] (the tanh form of gelu): ``z`` float32 [tokens, dim], ``table`` and
+    ``out`` [tokens, dim] of one element type."""
+    tokens, dim = out.shape
+    if tuple(z.shape) != (tokens, dim) or ids.numel() != tokens or at + dim > table.shape[1] or table.dtype != out.dtype:
+        raise KernelError("side_gate: shapes or types do not agree")
+    _check(library().ls_side_gate(
+        _dev(z, "z", torch.float32), _dev(ids, "ids", torch.int32), _dev(table, "table"), table.shape[1], int(at),
+        table.shape[0], _dev(out, "out"), _code(out), tokens, dim, _dev(err, "err", torch.int32), _stream()), "side_gate")
+
+
 def _rows(t: torch.Tensor, name: str) -> tuple[int, int]:
     """(pointer, row pitch in elements) of a 2-D operand whose rows are contiguous: a whole
     tensor, or a view of some columns of one."""
@@ -527,9 +543,11 @@ def _slopes(slopes, nq: int) -> int:
 
 
 def attention_tile(q, pages, out, part_acc, part_ml, work, n_work, block_table, nq, nkv, d,
-                   window, scale, err, slopes=None, log_rates=None, sinks=None, softcap: float = 0.0) -> None:
+                   window, scale, err, slopes=None, log_rates=None, sinks=None, softcap: float = 0.0,
+                   keep_first: int = 0) -> None:
     """``window`` > 0: a query reads the last ``window`` positions; < 0: the positions of its own chunk of
-    ``-window`` positions, chunks counted from position 0; 0: every earlier position.  ``softcap`` > 0: the scaled
+    ``-window`` positions, chunks counted from position 0; 0: every earlier position.  ``keep_first``: the first so
+    many positions are read besides, wherever the window is.  ``softcap`` > 0: the scaled
     score becomes softcap tanh(score / softcap) before any bias.  ``slopes`` (float32 [nq] or None): slopes[head] x (key position - query position) is added
     to every score; with ``log_rates`` [nq] as well, slopes[head] x ln(1 + log_rates[head] x (query
     position - key position)) is taken off instead.  ``sinks`` [nq]: exp(sinks[head]) is one more
@@ -539,19 +557,19 @@ def attention_tile(q, pages, out, part_acc, part_ml, work, n_work, block_table, 
         _dev(q, "q"), _dev(pages, "pages", q.dtype), _opt(out, "out", q.dtype),
         _opt(part_acc, "part_acc", torch.float32), _opt(part_ml, "part_ml", torch.float32), _code(q),
         _dev(work, "work", torch.int32), n_work, _dev(block_table, "block_table", torch.int32),
-        block_table.shape[-1], nq, nkv, d, pages.shape[3], pages.shape[0], int(window), float(scale), float(softcap),
-        _slopes(slopes, nq), _slopes(log_rates, nq), _slopes(sinks, nq), _dev(err, "err", torch.int32),
+        block_table.shape[-1], nq, nkv, d, pages.shape[3], pages.shape[0], int(window), int(keep_first), float(scale),
+        float(softcap), _slopes(slopes, nq), _slopes(log_rates, nq), _slopes(sinks, nq), _dev(err, "err", torch.int32),
         _stream()), "attention_tile")
 
 
 def attention_decode(q, pages, part_acc, part_ml, work, n_work, block_table, nq, nkv, d, window,
-                     scale, err, slopes=None, log_rates=None, softcap: float = 0.0) -> bool:
+                     scale, err, slopes=None, log_rates=None, softcap: float = 0.0, keep_first: int = 0) -> bool:
     """Returns False (and launches nothing) for shapes the decode kernel does not take."""
     status = library().ls_attention_decode(
         _dev(q, "q"), _dev(pages, "pages", q.dtype), _dev(part_acc, "part_acc", torch.float32),
         _dev(part_ml, "part_ml", torch.float32), _code(q), _dev(work, "work", torch.int32), n_work,
         _dev(block_table, "block_table", torch.int32), block_table.shape[-1], nq, nkv, d,
-        pages.shape[3], pages.shape[0], int(window), float(scale), float(softcap), _slopes(slopes, nq),
+        pages.shape[3], pages.shape[0], int(window), int(keep_first), float(scale), float(softcap), _slopes(slopes, nq),
         _slopes(log_rates, nq), _dev(err, "err", torch.int32), _stream())
     if status == -2:
         return False
@@ -560,12 +578,12 @@ def attention_decode(q, pages, part_acc, part_ml, work, n_work, block_table, nq,
 
 
 def attention_decode_mma(q, pages, part_acc, part_ml, work, n_work, block_table, nq, nkv, d, window,
-                         scale, err, slopes=None, log_rates=None) -> bool:
+                         scale, err, slopes=None, log_rates=None, softcap: float = 0.0, keep_first: int = 0) -> bool:
     """Decode attention on mma.sync with TMA-fed pages (csrc/attention_decode_mma.cu): bfloat16,
     head size 64 or 128, groups up to 16; ``slopes`` and ``log_rates`` together: the bias that grows
-    with the logarithm of the distance (see ``attention_tile``).  Returns False (nothing launched)
-    otherwise."""
-    if (slopes is None) != (log_rates is None):
+    with the logarithm of the distance; ``softcap`` (not beside that bias) and ``keep_first`` as in
+    ``attention_tile``.  Returns False (nothing launched) otherwise."""
+    if (slopes is None) != (log_rates is None) or (softcap and log_rates is not None):
         return False
     if q.dtype != torch.bfloat16 or not USE_TENSOR_CORES[0]:
         return False
@@ -573,8 +591,8 @@ def attention_decode_mma(q, pages, part_acc, part_ml, work, n_work, block_table,
         _dev(q, "q"), _dev(pages, "pages", q.dtype), _dev(part_acc, "part_acc", torch.float32),
         _dev(part_ml, "part_ml", torch.float32), _dev(work, "work", torch.int32), n_work,
         _dev(block_table, "block_table", torch.int32), block_table.shape[-1], nq, nkv, d,
-        pages.shape[3], pages.shape[0], int(window), float(scale), _slopes(slopes, nq), _slopes(log_rates, nq),
-        _dev(err, "err", torch.int32), _stream())
+        pages.shape[3], pages.shape[0], int(window), int(keep_first), float(scale), float(softcap), _slopes(slopes, nq),
+        _slopes(log_rates, nq), _dev(err, "err", torch.int32), _stream())
     if status == -2:
         return False
     _check(status, "attention_decode_mma")
@@ -586,11 +604,11 @@ def attention_prefill_tc_tile_tokens() -> int:
 
 
 def attention_prefill_tc(q, pages, out, work, n_work, block_table, nq, nkv, d, window, scale, err,
-                         slopes=None, log_rates=None, sinks=None, softcap: float = 0.0) -> bool:
+                         slopes=None, log_rates=None, sinks=None, softcap: float = 0.0, keep_first: int = 0) -> bool:
     """Attention of prompt portions on tcgen05 (csrc/attention_prefill_tc.cu): bfloat16, head
     size 64 or 128, work items of up to 128 tokens; ``slopes`` with ``log_rates`` (the bias that
     grows with the logarithm of the distance), ``slopes`` alone (the bias linear in the distance), ``softcap`` and
-    ``sinks`` as in ``attention_tile``.  Returns False (nothing launched) for anything else."""
+    ``sinks`` and ``keep_first`` as in ``attention_tile``.  Returns False (nothing launched) for anything else."""
     if log_rates is not None and (slopes is None or softcap):
         return False
     if q.dtype != torch.bfloat16 or not USE_TENSOR_CORES[0]:
@@ -598,7 +616,7 @@ def attention_prefill_tc(q, pages, out, work, n_work, block_table, nq, nkv, d, w
     status = library("tc").ls_attention_prefill_tc(
         _dev(q, "q"), _dev(pages, "pages", q.dtype), _dev(out, "out", q.dtype), q.shape[0],
         _dev(work, "work", torch.int32), n_work, _dev(block_table, "block_table", torch.int32),
-        block_table.shape[-1], nq, nkv, d, pages.shape[3], pages.shape[0], int(window), float(scale),
+        block_table.shape[-1], nq, nkv, d, pages.shape[3], pages.shape[0], int(window), int(keep_first), float(scale),
         _slopes(slopes, nq), _slopes(log_rates, nq), _slopes(sinks, nq), float(softcap), _dev(err, "err", torch.int32), _stream())
     if status in (-2, -3):
         return False
@@ -763,18 +781,21 @@ def gemm_nt(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, epilogue: int = E
 # library "seq": heads of unequal sizes, mixers with a carried state, routed experts
 # ---------------------------------------------------------------------------
 
-RULE_DELTA, RULE_WKV, RULE_GLA = 0, 1, 2
+RULE_DELTA, RULE_WKV, RULE_GLA, RULE_DELTA_HEAD, RULE_MLSTM = 0, 1, 2, 3, 4
 
 
 def qkv_finish(qkv, q_out, pages, q_gain, k_gain, cos, sin, positions, token_req, block_table, nq: int, nkv: int,
                d: int, dv: int, pad: int, rot_dim: int, eps: float, whole_projection: bool, has_kv: bool,
-               write_cache: bool, err, bias=None, q_temp=None) -> None:
+               write_cache: bool, err, bias=None, q_temp=None, interleaved: bool = False, v_other=None,
+               v_mix=None) -> None:
     """Finishes a projection ``qkv`` [tokens, nq*d (+ nkv*d + nkv*dv)]: RMSNorm of q and of k (over
     the whole projection, or per head), rotation of the first ``rot_dim`` elements of each head,
     queries to ``q_out`` [tokens, nq*pad] and keys and values into ``pages``
     [num_pages, 2, nkv, page_size, pad], padded with zeros (csrc/heads_wide.cu).  ``bias`` (one
     element per column of ``qkv``, or None) is added first; ``q_temp`` = (coef, every): the query at
-    position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+    position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  ``interleaved``: neighbouring elements
+    are rotated as pairs instead of the halves.  ``v_other`` ([tokens, nkv*dv], possibly columns of a wider tensor)
+    and ``v_mix`` (one float32): v <- (1 - v_mix) v + v_mix v_other before the values are written."""
     tokens = qkv.shape[0]
     cols = nq * d + (nkv * (d + dv) if has_kv else 0)
     if qkv.shape[1] != cols or q_out.shape != (tokens, nq * pad) or q_out.dtype != qkv.dtype:
@@ -797,6 +818,11 @@ def qkv_finish(qkv, q_out, pages, q_gain, k_gain, cos, sin, positions, token_req
     if bias is not None and bias.numel() != cols:
         raise KernelError("qkv_finish: the bias does not match the projection")
     coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 1)
+    vp, v_ld = (0, 0)
+    if v_other is not None:
+        if v_other.dtype != qkv.dtype or tuple(v_other.shape) != (tokens, nkv * dv) or v_mix is None or v_mix.numel() != 1:
+            raise KernelError("qkv_finish: the values to mix in do not match")
+        vp, v_ld = _rows(v_other, "v_other")
     _check(library("seq").ls_qkv_finish(
         _dev(qkv, "qkv"), qkv.shape[1], _dev(q_out, "q_out"), _opt(pages if write_cache else None, "pages"),
         _code(qkv), _opt(q_gain, "q_gain"), _opt(k_gain, "k_gain"), _code(gains[0]) if gains else F32,
@@ -805,7 +831,8 @@ def qkv_finish(qkv, q_out, pages, q_gain, k_gain, cos, sin, positions, token_req
         _dev(block_table, "block_table", torch.int32), block_table.shape[-1], tokens, nq, nkv, d, dv, pad, rot_dim,
         page_size, num_pages, cos.shape[0] if rot_dim else 0, float(eps), 2 if whole_projection else 1,
         1 if has_kv else 0, 1 if write_cache else 0, _opt(bias, "bias"), _code(bias) if bias is not None else F32,
-        coef, every, _dev(err, "err", torch.int32), _stream()), "qkv_finish")
+        coef, every, 1 if interleaved else 0, vp, v_ld, _opt(v_mix if vp else None, "v_mix", torch.float32),
+        _dev(err, "err", torch.int32), _stream()), "qkv_finish")
 
 
 def latent_finish(proj, q_out, pages, gain, cos, sin, positions, token_req, block_table, heads: int, d: int, dr: int,
@@ -876,18 +903,20 @@ def find_portions(token_slot, out, cap: int, err) -> None:
 
 
 def delta_prep(proj, conv_w, dt_bias, a_log, state, token_slot, qkv, decay, beta, heads: int, groups: int, dk: int,
-               dv: int, taps: int, unit_eps: float) -> None:
+               dv: int, taps: int, unit_eps: float, gates=None) -> None:
     """What lies between the projections and the gated delta rule, a token a block: causal
     convolution (carried inputs from ``state``) and silu of q, k, v, unit q and k (q scaled),
     beta = sigmoid of its column, and the decay per key channel, made in place from the output
     of its low-rank map: ``decay`` <- exp(-exp(a_log[head]) softplus(decay + dt_bias)).  float32 out.
-    ``proj`` [tokens, >= 2 G dk + H dv + H]."""
+    ``proj`` [tokens, >= 2 G dk + H dv + H].  With ``gates`` (float32 [tokens, 2 H]: the logits of beta, then those
+    of one decay per head) beta comes from there and ``decay`` [tokens, H] is written only."""
     f32 = torch.float32
     _check(library("seq").ls_delta_prep(
         _dev(proj, "proj"), proj.shape[1], _code(proj), _dev(conv_w, "conv_w", f32), _dev(dt_bias, "dt_bias", f32),
         _dev(a_log, "a_log", f32), _dev(state, "state", f32), state.shape[1],
         _dev(token_slot, "token_slot", torch.int32), _dev(qkv, "qkv", f32), _dev(decay, "decay", f32),
-        _dev(beta, "beta", f32), proj.shape[0], heads, groups, dk, dv, taps, float(unit_eps), _stream()), "delta_prep")
+        _dev(beta, "beta", f32), _opt(gates, "gates", f32), proj.shape[0], heads, groups, dk, dv, taps, float(unit_eps),
+        _stream()), "delta_prep")
 
 
 def double_exp_decay(z, bias) -> None:
@@ -916,13 +945,21 @@ def tanh_rows(x) -> None:
 
 def state_rule(rule: int, dtype, portions, max_portions: int, state, in_a, in_b, in_v, decay, beta, bonus, out,
                carry_src, carry_width: int, carry_rows: int, heads: int, groups: int, dk: int, dv: int,
-               out_scale: float = 1.0, decay_fixed: bool = False) -> None:
+               out_scale: float = 1.0, decay_fixed: bool = False, gate_bias=None, gate_cap: float = 0.0) -> None:
     """(``decay_fixed``: ``decay`` is one row [heads dk] that serves every token.)  Walks every portion of the step through a state rule (RULE_DELTA, RULE_WKV, RULE_GLA), reading and
     writing ``state[slot]`` (float32: the matrix state, then the carried inputs).  RULE_GLA (S <- diag(decay) S
     + k v^T, o = out_scale S^T q) carries nothing else; its ``in_a``, ``in_b``, ``in_v`` (q, k, v in the engine's
-    type) may be views of columns of one wider tensor."""
+    type) may be views of columns of one wider tensor.  RULE_DELTA_HEAD is RULE_DELTA with ``decay`` [tokens, heads].
+    RULE_MLSTM takes q, k, v as RULE_GLA does and the logits of its gates as ``decay`` [tokens, 2 heads] with ``gate_bias``
+    [2 heads] and ``gate_cap``; its state is [heads, dk + 1, dv + 1] and ``out`` [tokens, heads (dv + 2)]: S^T q, n . q and
+    exp(-m), which ``head_rms_gate`` takes as ``normalized``."""
     in_ld = 0
-    if rule == RULE_GLA:
+    if rule == RULE_MLSTM and (out.shape[1] != heads * (dv + 2) or state.shape[1] != heads * (dk + 1) * (dv + 1)
+                               or gate_bias is None or gate_bias.numel() != 2 * heads or decay.shape[1] != 2 * heads):
+        raise KernelError("state_rule: the read-out, the state or the gates do not match")
+    if rule == RULE_DELTA_HEAD and decay.shape[1] != heads:
+        raise KernelError("state_rule: one decay per head")
+    if rule in (RULE_GLA, RULE_MLSTM):
         (pa, in_ld), (pb, ldb), (pv, ldv) = _rows(in_a, "in_a"), _rows(in_b, "in_b"), _rows(in_v, "in_v")
         if not (in_ld == ldb == ldv) or not (in_a.dtype == in_b.dtype == in_v.dtype == dtype):
             raise KernelError("state_rule: q, k and v must be columns of rows of one pitch, in the engine's type")
@@ -934,14 +971,18 @@ def state_rule(rule: int, dtype, portions, max_portions: int, state, in_a, in_b,
         _dev(decay, "decay", torch.float32), _opt(beta, "beta", torch.float32), _opt(bonus, "bonus", torch.float32),
         _dev(out, "out", torch.float32), _opt(carry_src, "carry_src", dtype),
         carry_src.shape[1] if carry_src is not None else 0, carry_width,
-        carry_rows, heads, groups, dk, dv, in_ld, float(out_scale), 0 if decay_fixed else -1, _stream()), "state_rule")
+        carry_rows, heads, groups, dk, dv, in_ld, float(out_scale), 0 if decay_fixed else -1,
+        _opt(gate_bias, "gate_bias", torch.float32), float(gate_cap), _stream()), "state_rule")
 
 
 def head_rms_gate(o, gain, gate_f32, gate_x, out, heads: int, dv: int, gain_shared: bool, eps: float,
-                  gate_logit: bool = False) -> None:
+                  gate_logit: bool = False, normalized: bool = False) -> None:
     """out = o / rms_per_head(o) * gain * gate, where the gate is ``gate_f32`` as it is (or its
-    sigmoid, ``gate_logit``), or silu(``gate_x``); ``gate_x`` may be a view of some columns of a
-    wider tensor."""
+    sigmoid, ``gate_logit``), or silu(``gate_x``) (or its sigmoid, ``gate_logit``); ``gate_x`` may be a view of some
+    columns of a wider tensor.  ``normalized``: every head of ``o`` has two more elements, a and b, and is first
+    divided by max(|a|, b) + 1e-6."""
+    if o.shape[1] != heads * (dv + 2 if normalized else dv):
+        raise KernelError("head_rms_gate: the read-out does not match the heads")
     gate_p, gate_ld = (0, 0)
     if gate_x is not None:
         if gate_x.dtype != out.dtype or gate_x.shape != (o.shape[0], heads * dv):
@@ -950,7 +991,8 @@ def head_rms_gate(o, gain, gate_f32, gate_x, out, heads: int, dv: int, gain_shar
     _check(library("seq").ls_head_rms_gate(
         _dev(o, "o", torch.float32), _dev(gain, "gain", torch.float32), _opt(gate_f32, "gate_f32", torch.float32),
         gate_p, _dev(out, "out"), _code(out), o.shape[0], heads, dv,
-        1 if gain_shared else 0, 1 if gate_logit else 0, float(eps), gate_ld, _stream()), "head_rms_gate")
+        1 if gain_shared else 0, 1 if gate_logit else 0, float(eps), gate_ld, 1 if normalized else 0, _stream()),
+        "head_rms_gate")
 
 
 def unit_gates(proj, x_at: int, x_bias, conv_w, conv_b, state, token_slot, w_r, w_i, b_r, b_i, rate, a_out, b_out,

@@ -30,6 +30,11 @@ Further parameters, for designs that differ from that one:
 - ``chunk``: a query sees the earlier keys of its own chunk of ``chunk`` positions only, chunks counted from
   position 0 of the sequence (the kernels take it as a negative window; every page is kept).
 - ``softcap``: the scaled score becomes softcap tanh(score / softcap) before any bias is taken off (CUDA-core kernels).
+- ``keep_first``: the first so many positions stay visible wherever the window is (their pages are kept).
+- ``qk_norm_gain`` False: the norm of q and k has no gain (a norm per head without a gain commutes with the rotation).
+- ``value_mix`` "first" / "later": layers whose values are mixed.  The first such layer leaves its values of the step's
+  tokens, as projected, with the step; a later one caches (1 - mix) v + mix v_first with a number ``mix`` of its own
+  (``names``: ``v_mix``).
 - ``sink``: a learned number per query head (``names``: ``sink``) whose exponential is one more term
   of the softmax's denominator; it has no key and no value.
 """
@@ -46,7 +51,7 @@ from .norm import NormedRows
 _DEFAULT_NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
                   "q_norm": "q_norm.weight", "k_norm": "k_norm.weight",
                   "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "o_bias": "o_proj.bias",
-                  "r1": "r1", "r2": "r2", "sink": "sink"}
+                  "r1": "r1", "r2": "r2", "sink": "sink", "v_mix": "v_mix"}
 
 
 def _f32(t: torch.Tensor) -> torch.Tensor:
@@ -56,38 +61,41 @@ def _f32(t: torch.Tensor) -> torch.Tensor:
 class ScoreExtras:
     """What the attention kernels add to plain scaled scores: a bias that grows with the distance
     of key and query (``slopes`` alone: linear; with ``log_rates``: logarithmic) and sinks.  The
-    tensor-core kernel of prompt portions knows all of them; that of decoded tokens the logarithmic bias (a linear
-    bias or a cap keeps decoded tokens on the CUDA-core kernels)."""
+    tensor-core kernel of prompt portions knows all of them; that of decoded tokens the logarithmic bias or a cap (a
+    linear bias keeps decoded tokens on the CUDA-core kernels)."""
 
     def __init__(self, slopes=None, log_rates=None, sinks=None, softcap: float = 0.0):
         self.slopes, self.log_rates, self.sinks, self.softcap = slopes, log_rates, sinks, float(softcap or 0.0)
 
     def tensor_cores(self) -> bool:
         """Whether the tensor-core kernel of decoded tokens knows these extras (that of prompt portions knows all)."""
-        return (self.slopes is None or self.log_rates is not None) and not self.softcap
+        return self.slopes is None or (self.log_rates is not None and not self.softcap)
 
 
-def attend(rt: Runtime, q, ctx, cache, nq: int, nkv: int, d: int, window: int, scale: float, exact: bool,
+def attend(rt: Runtime, q, ctx, cache, nq: int, nkv: int, d: int, mask, scale: float, exact: bool,
            extras: ScoreExtras) -> torch.Tensor:
     """Causal attention of the step's queries ``q`` [tokens, nq d] over a layer's pages (heads of one
     size ``d``): prompt portions by tiles, single tokens by splits and a fold.  Returns [tokens, nq d]
     in the engine's type.  ``exact``: every row takes the tile kernel, so that a row's bits do not
-    depend on whether it was decoded or part of a prompt.  ``window`` < 0: chunks of -window positions."""
+    depend on whether it was decoded or part of a prompt.  ``mask``: a window (0: none, < 0: chunks of -window
+    positions), or a pair of a window and the number of first positions that stay visible."""
     t = q.shape[0]
+    window, keep = mask if isinstance(mask, tuple) else (mask, 0)
     tensor_core_attention = not exact and extras.tensor_cores()
     attn = rt.rows(t, nq * d)
     plan, done = None, False
     if not exact and d in (64, 128):
-        plan = ctx.attention_plan(window, K.attention_prefill_tc_tile_tokens())
+        plan = ctx.attention_plan(mask, K.attention_prefill_tc_tile_tokens())
         done = not plan.n_tile or K.attention_prefill_tc(
             q, cache.pages, attn, plan.tile_work, plan.n_tile, cache.block_table, nq, nkv, d,
-            window, scale, rt.err, extras.slopes, extras.log_rates, extras.sinks, softcap=extras.softcap)
+            window, scale, rt.err, extras.slopes, extras.log_rates, extras.sinks, softcap=extras.softcap,
+            keep_first=keep)
     if not done:
-        plan = ctx.attention_plan(window)
+        plan = ctx.attention_plan(mask)
         if plan.n_tile:
             K.attention_tile(q, cache.pages, attn, None, None, plan.tile_work, plan.n_tile,
                              cache.block_table, nq, nkv, d, window, scale, rt.err, extras.slopes,
-                             extras.log_rates, extras.sinks, softcap=extras.softcap)
+                             extras.log_rates, extras.sinks, softcap=extras.softcap, keep_first=keep)
     if plan.n_split:
         part_acc = rt.rows(plan.n_slots, nq, d, dtype=torch.float32)
         part_ml = rt.rows(plan.n_slots, nq, 2, dtype=torch.float32)
@@ -95,15 +103,17 @@ def attend(rt: Runtime, q, ctx, cache, nq: int, nkv: int, d: int, window: int, s
         if tensor_core_attention:
             done = K.attention_decode_mma(q, cache.pages, part_acc, part_ml, plan.split_work,
                                           plan.n_split, cache.block_table, nq, nkv, d, window,
-                                          scale, rt.err, extras.slopes, extras.log_rates)
+                                          scale, rt.err, extras.slopes, extras.log_rates, softcap=extras.softcap,
+                                          keep_first=keep)
         if not done and not exact:
             done = K.attention_decode(q, cache.pages, part_acc, part_ml, plan.split_work,
                                       plan.n_split, cache.block_table, nq, nkv, d, window,
-                                      scale, rt.err, extras.slopes, extras.log_rates, softcap=extras.softcap)
+                                      scale, rt.err, extras.slopes, extras.log_rates, softcap=extras.softcap,
+                                      keep_first=keep)
         if not done:
             K.attention_tile(q, cache.pages, None, part_acc, part_ml, plan.split_work,
                              plan.n_split, cache.block_table, nq, nkv, d, window,
-                             scale, rt.err, extras.slopes, extras.log_rates, softcap=extras.softcap)
+                             scale, rt.err, extras.slopes, extras.log_rates, softcap=extras.softcap, keep_first=keep)
         K.attention_combine(part_acc, part_ml, attn, plan.combine_items, plan.n_combine, nq, d, extras.sinks)
     return attn
 
@@ -116,7 +126,7 @@ class GQAttention(Mixer):
     def __init__(self, hidden_size, num_heads, num_kv_heads, head_dim, scale, window, qk_norm_eps,
                  position: PositionEncoding, runtime: Runtime, value_dim=None, qk_norm_scope="head",
                  borrows_kv=False, names=None, bias=False, q_temp=None, score_bias=None, sink=False,
-                 value_from_key=False, chunk=0, softcap=0.0):
+                 value_from_key=False, chunk=0, softcap=0.0, keep_first=0, qk_norm_gain=True, value_mix=None):
         if num_heads % num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
         if qk_norm_scope not in ("head", "projection"):
@@ -133,14 +143,21 @@ class GQAttention(Mixer):
             raise ValueError("value_from_key: value heads have the size of key heads, and the layer projects its own keys without biases")
         if self.chunk < 0 or (self.chunk and window):
             raise ValueError("chunk must be positive, and a layer has a window or chunks, not both")
+        self.keep_first, self.qk_norm_gain, self.value_mix = int(keep_first or 0), bool(qk_norm_gain), value_mix
+        if self.keep_first < 0 or (self.keep_first and not window):
+            raise ValueError("keep_first goes with a window")
+        if value_mix not in (None, "first", "later") or (value_mix and self.borrows):
+            raise ValueError(f"value_mix must be first, later or absent, in a layer with values of its own; got {value_mix!r}")
+        if not self.qk_norm_gain and self.scope != "head":
+            raise ValueError("a norm of q and k without a gain is one per head")
         self.q_temp = (float(q_temp["coef"]), int(q_temp["every"])) if q_temp else None
         if self.q_temp is not None and self.q_temp[1] <= 0:
             raise ValueError("q_temp.every must be positive")
         # the general finishing kernel (norm over the projection, heads padded to one size, biases,
-        # a query temperature) where the design asks for any of this; else the per-head kernels
-        # and the fused products
+        # a query temperature, values to mix) where the design asks for any of this; else the per-head
+        # kernels and the fused products
         self.wide = self.scope == "projection" or self.dv != self.d or self.borrows or self.d % 16 != 0 \
-            or self.bias or self.q_temp is not None
+            or self.bias or self.q_temp is not None or value_mix is not None
         self.pad = -(-max(self.d, self.dv) // 16) * 16 if self.wide else self.d
         if self.pad % 16 or not 16 <= self.pad <= 256:
             raise ValueError(
@@ -148,17 +165,18 @@ class GQAttention(Mixer):
         self.names = dict(_DEFAULT_NAMES)
         self.names.update(names or {})
         self.scale, self.window = float(scale), int(window or 0)
-        self.mask = -self.chunk if self.chunk else self.window     # what the attention kernels and plans are given
+        # what the attention kernels and plans are given
+        self.mask = -self.chunk if self.chunk else (self.window, self.keep_first) if self.keep_first else self.window
         self.qk_norm_eps = qk_norm_eps
         self.position, self.rt = position, runtime
-        self.w_qkv = self.w_o = self.q_gain = self.k_gain = self.qkv_bias = self.o_bias = None
+        self.w_qkv = self.w_o = self.q_gain = self.k_gain = self.qkv_bias = self.o_bias = self.v_mix = None
         self.extras = ScoreExtras()
         # in float32 every row takes the tile kernel, so that a row's bits do not
         # depend on whether it was decoded or part of a prompt
         self.exact = runtime.dtype == torch.float32
 
     def cache_need(self):
-        return CacheNeed("paged_kv", kv_heads=self.nkv, head_dim=self.pad, window=self.window)
+        return CacheNeed("paged_kv", kv_heads=self.nkv, head_dim=self.pad, window=self.window, keep_first=self.keep_first)
 
     def attention_windows(self):
         return {self.mask}
@@ -172,7 +190,7 @@ class GQAttention(Mixer):
             specs[n["k"]] = WeightSpec((self.nkv * self.d, self.h))
             if not self.value_from_key:
                 specs[n["v"]] = WeightSpec((self.nkv * self.dv, self.h))
-        if self.qk_norm_eps is not None:
+        if self.qk_norm_eps is not None and self.qk_norm_gain:
             specs[n["q_norm"]] = WeightSpec((self.nq * self.d if whole else self.d,), "gain")
             if not self.borrows:
                 specs[n["k_norm"]] = WeightSpec((self.nkv * self.d if whole else self.d,), "gain")
@@ -189,6 +207,8 @@ class GQAttention(Mixer):
             specs[n["r2"]] = WeightSpec((self.nq,), "gain", ("uniform", 0.05, 1.0))
         if self.sink:
             specs[n["sink"]] = WeightSpec((self.nq,), "gain", ("normal", 0.0, 1.0))
+        if self.value_mix == "later":
+            specs[n["v_mix"]] = WeightSpec((), "gain", ("uniform", 0.0, 1.0))
         return specs
 
     def bind(self, tensors):
@@ -215,7 +235,12 @@ class GQAttention(Mixer):
             parts = [tensors[n["q_bias"]]] if self.borrows else [tensors[n[k]] for k in ("q_bias", "k_bias", "v_bias")]
             self.qkv_bias = _f32(torch.cat([p.reshape(-1) for p in parts]))
             self.o_bias = _f32(tensors[n["o_bias"]]) if self.output_biased else None
-        if self.qk_norm_eps is not None:
+        if self.value_mix == "later":
+            self.v_mix = _f32(tensors[n["v_mix"]].reshape(1))
+        if self.qk_norm_eps is not None and not self.qk_norm_gain:
+            self.q_gain = torch.ones(self.d, dtype=torch.float32, device=self.w_qkv.device)
+            self.k_gain = None if self.borrows else self.q_gain
+        elif self.qk_norm_eps is not None:
             self.q_gain = tensors[n["q_norm"]]
             self.k_gain = None if self.borrows else tensors[n["k_norm"]]
 
@@ -226,11 +251,17 @@ class GQAttention(Mixer):
             x.linear(self.w_qkv, qkv, K.EPILOGUE_STORE, self.rt.err)
         else:
             K.gemm_nt(x, self.w_qkv, qkv, err=self.rt.err)
+        v_other = None
+        if self.value_mix == "first":
+            ctx._first_values = qkv[:, (self.nq + self.nkv) * self.d:]       # as projected; kept while the step runs
+        elif self.value_mix == "later":
+            v_other = ctx._first_values
         q = self.rt.rows(t, self.nq * self.pad)
         K.qkv_finish(qkv, q, cache.pages, self.q_gain, self.k_gain, cos, sin, ctx.positions, ctx.token_slot,
                      cache.block_table, self.nq, self.nkv, self.d, self.dv, self.pad, rot_dim,
                      self.qk_norm_eps or 0.0, self.scope == "projection", not self.borrows,
-                     bool(cache.writes) and not self.borrows, self.rt.err, bias=self.qkv_bias, q_temp=self.q_temp)
+                     bool(cache.writes) and not self.borrows, self.rt.err, bias=self.qkv_bias, q_temp=self.q_temp,
+                     interleaved=bool(rot_dim and self.position.rotary_interleaved), v_other=v_other, v_mix=self.v_mix)
         return q
 
     def output_bias(self):
@@ -242,8 +273,6 @@ class GQAttention(Mixer):
         rot = self.position.rotary()
         cos, sin, rot_dim = rot if rot is not None else (None, None, 0)
         if self.wide:
-            if rot_dim and self.position.rotary_interleaved:
-                raise ValueError("rotation of neighbouring pairs is not available with padded heads")
             q = self._project_wide(x, ctx, cache, t, cos, sin, rot_dim)
             return self._attend(q, ctx, cache, residual, t, overwrite)
         q = self.rt.rows(t, nq * d)
@@ -287,4 +316,5 @@ def _build(spec, runtime, position=None, **_):
                        borrows_kv=spec.get("borrows_kv", False), names=spec.get("names"),
                        bias=spec.get("bias", False), q_temp=spec.get("q_temp"), score_bias=spec.get("score_bias"),
                        sink=spec.get("sink", False), value_from_key=spec.get("value_from_key", False),
-                       chunk=spec.get("chunk", 0), softcap=spec.get("softcap", 0.0))
+                       chunk=spec.get("chunk", 0), softcap=spec.get("softcap", 0.0), keep_first=spec.get("keep_first", 0),
+                       qk_norm_gain=spec.get("qk_norm_gain", True), value_mix=spec.get("value_mix"))

@@ -43,7 +43,7 @@ class CacheNeed:
     """What a mixer keeps between steps.
 
     kind "paged_kv": keys and values of ``kv_heads`` x ``head_dim`` per token in
-    pages; ``window`` > 0 means only the last ``window`` positions are read, so
+    pages; ``window`` > 0 means only the last ``window`` positions (and the first ``keep_first``) are read, so
     pages behind it can be given back.  kind "state": one tensor of
     ``state_shape`` per request, of fixed size, in a slot.  kind "several": the needs ``parts``
     side by side (a mixer made of several, each with a cache of its own); the mixer gets a
@@ -54,24 +54,26 @@ class CacheNeed:
     kv_heads: int = 0
     head_dim: int = 0
     window: int = 0
+    keep_first: int = 0
     state_shape: tuple[int, ...] = ()
     state_dtype: torch.dtype = torch.float32
     parts: tuple = ()
 
     def widened(self, reader: "CacheNeed | None") -> "CacheNeed":
         """This need, kept for as long as ``reader`` (a layer that reads the entry without
-        writing it) also asks: the longer of the two windows, 0 standing for every key."""
+        writing it) also asks: the longer of the two windows, 0 standing for every key, and the more of the first keys."""
         if reader is None or self.kind != "paged_kv":
             return self
         if (reader.kind, reader.kv_heads, reader.head_dim) != (self.kind, self.kv_heads, self.head_dim):
             raise ValueError("a layer reads a cache entry whose keys and values do not have its sizes")
         window = 0 if (self.window == 0 or reader.window == 0) else max(self.window, reader.window)
-        return self if window == self.window else CacheNeed(
-            self.kind, kv_heads=self.kv_heads, head_dim=self.head_dim, window=window)
+        keep = max(self.keep_first, reader.keep_first) if window else 0
+        return self if (window, keep) == (self.window, self.keep_first) else CacheNeed(
+            self.kind, kv_heads=self.kv_heads, head_dim=self.head_dim, window=window, keep_first=keep)
 
     def group_key(self):
         if self.kind == "paged_kv":
-            return ("paged_kv", self.kv_heads, self.head_dim, self.window)
+            return ("paged_kv", self.kv_heads, self.head_dim, self.window, self.keep_first)
         return ("state", tuple(self.state_shape), str(self.state_dtype))
 
 
@@ -85,6 +87,8 @@ class Runtime:
     max_positions: int
     err: torch.Tensor            # int32[2] device error word
     options: dict = field(default_factory=dict)
+    # parts that several layers use (``ModelSpec.shared``), by name; there before the layers are built
+    shared: dict = field(default_factory=dict)
     # True while a step is recorded into a CUDA graph: buffers then have exactly the rows asked
     # for (they are kept for the graph's life, and their sizes never change).
     exact_sizes: bool = False
@@ -140,8 +144,8 @@ class Part:
     # inside its first product.  Parts that leave it False always get a tensor.
     accepts_normed_rows = False
 
-    def attention_windows(self) -> set[int]:
-        """Window sizes for which this part asks ``ctx.attention_plan``."""
+    def attention_windows(self) -> set:
+        """Masks (``engine.batch.mask_parts``) for which this part asks ``ctx.attention_plan``."""
         return set()
 
     def weight_specs(self) -> dict[str, WeightSpec]:
@@ -231,7 +235,7 @@ class Block(Part):
 # registries: (category, kind) -> builder(spec, runtime, **extra) -> Part
 # ---------------------------------------------------------------------------
 
-CATEGORIES = ("block", "mixer", "feed_forward", "norm", "position", "embedding", "head", "injection")
+CATEGORIES = ("block", "mixer", "feed_forward", "norm", "position", "embedding", "head", "injection", "table", "side")
 _BUILDERS: dict[tuple[str, str], Callable[..., Part]] = {}
 
 

@@ -2,7 +2,8 @@
 h += mixer(norm_a(h)); h += feed_forward(norm_b(h))  (LockStep: engine/model/qwen3.py:242-287).
 The names under which the layer's tensors are stored are parameters of the
 arrangement, so the same arrangement serves architectures that name them otherwise.
-A layer whose feed-forward is of kind "none" is its mixer alone.
+A layer whose feed-forward is of kind "none" is its mixer alone.  With ``LayerSpec.extra["side"]`` (a part of category
+``side``: an input of the layer besides the stream) that part adds its result to the stream last.
 
 "sandwich_norm": a norm after each sublayer as well as before it,
 h += norm_c(mixer(norm_a(h))); h += norm_d(feed_forward(norm_b(h))).  The norms after the sublayers are the
@@ -33,6 +34,7 @@ _DEFAULT_NAMES = {
     "mixer": "self_attn",
     "feed_forward_norm": "post_attention_layernorm",
     "feed_forward": "mlp",
+    "side": "side",
 }
 
 
@@ -48,6 +50,7 @@ class PreNormBlock(Block):
         if layer_spec.feed_forward.kind != "none":
             self.feed_forward_norm = build_part("norm", layer_spec.feed_forward_norm, runtime)
             self.feed_forward = build_part("feed_forward", layer_spec.feed_forward, runtime)
+        self.side = build_part("side", layer_spec.extra["side"], runtime) if "side" in layer_spec.extra else None
 
     def _children(self):
         return [(self.names[k], getattr(self, k)) for k in _DEFAULT_NAMES if getattr(self, k) is not None]
@@ -88,16 +91,20 @@ class PreNormBlock(Block):
     def _feed_forward(self, h, ctx, cache):
         self.feed_forward.forward(self._normed(self.feed_forward_norm, self.feed_forward, h), ctx, h)
 
+    def _side(self, h, ctx, cache):
+        self.side.forward(h, ctx)
+
     def steps(self):
         out = [(bool(self.mixer_norm.graph_safe and self.mixer.graph_safe and self.position.graph_safe), self._mix)]
         if self.feed_forward is not None:
             out.append((bool(self.feed_forward_norm.graph_safe and self.feed_forward.graph_safe), self._feed_forward))
+        if self.side is not None:
+            out.append((bool(self.side.graph_safe), self._side))
         return out
 
     def forward(self, h, ctx, cache):
-        self._mix(h, ctx, cache)
-        if self.feed_forward is not None:
-            self._feed_forward(h, ctx, cache)
+        for _, step in self.steps():
+            step(h, ctx, cache)
 
 
 @register_part("block", "pre_norm")

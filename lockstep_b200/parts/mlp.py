@@ -126,6 +126,39 @@ class GatedUnit(FeedForward):
         K.gemm_nt(act, self.w_down, residual, K.EPILOGUE_STORE if overwrite else K.EPILOGUE_RESIDUAL, err=self.rt.err)
 
 
+class PlainUnit(FeedForward):
+    """down(gelu_tanh(up(x))) without biases and without a gate; the activation is made in the first product's epilogue."""
+
+    graph_safe = True
+    accepts_normed_rows = True
+    can_overwrite = True
+
+    def __init__(self, hidden_size: int, intermediate_size: int, runtime: Runtime, names=None):
+        self.h, self.i, self.rt = int(hidden_size), int(intermediate_size), runtime
+        self.names = {"up": "up", "down": "down"}
+        self.names.update(names or {})
+        self.w_up = self.w_down = None
+
+    def weight_specs(self):
+        return {self.names["up"]: WeightSpec((self.i, self.h)), self.names["down"]: WeightSpec((self.h, self.i))}
+
+    def bind(self, tensors):
+        self.w_up, self.w_down = tensors[self.names["up"]], tensors[self.names["down"]]
+
+    def forward(self, x, ctx, residual, overwrite=False):
+        act = self.rt.rows(residual.shape[0], self.i)
+        if isinstance(x, NormedRows):
+            x.linear(self.w_up, act, K.EPILOGUE_GELU, self.rt.err)
+        else:
+            K.gemm_nt(x, self.w_up, act, K.EPILOGUE_GELU, err=self.rt.err)
+        K.gemm_nt(act, self.w_down, residual, K.EPILOGUE_STORE if overwrite else K.EPILOGUE_RESIDUAL, err=self.rt.err)
+
+
+@register_part("feed_forward", "plain_unit")
+def _build_plain_unit(spec, runtime, **_):
+    return PlainUnit(spec["hidden_size"], spec["intermediate_size"], runtime, names=spec.get("names"))
+
+
 @register_part("feed_forward", "gated_unit")
 def _build_gated_unit(spec, runtime, **_):
     return GatedUnit(spec["hidden_size"], spec["intermediate_size"], spec.get("activation", "gelu_tanh"), runtime,

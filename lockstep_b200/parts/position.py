@@ -8,8 +8,10 @@ smaller than the head size; the dimensions past it are left as they are.
 (the YaRN scheme): with f_i = theta^(-2i/dim) and dim(t) = dim ln(original / (2 pi t)) / (2 ln theta),
 lo = max(floor(dim(fast)), 0), hi = min(ceil(dim(slow)), dim - 1), ramp_i = clamp((i - lo) / max(hi - lo,
 0.001), 0, 1), the frequency is f_i / factor * ramp_i + f_i (1 - ramp_i), and cosines and sines are
-multiplied by 0.1 ln(factor) + 1.  Without ``scaling`` it is the plain rotation.  ``interleaved``: a
-pair is elements (2i, 2i + 1) instead of (i, i + dim / 2).
+multiplied by 0.1 ln(factor) + 1.  ``scaling`` with ``kind`` "wavelength" (the scheme of Llama 3.1) instead: with
+wavelength l_i = 2 pi / f_i, f_i stays where l_i < original / high, is divided by ``factor`` where l_i > original / low,
+and is (1 - s) f_i / factor + s f_i with s = (original / l_i - low) / (high - low) between the two.  Without ``scaling``
+it is the plain rotation.  ``interleaved``: a pair is elements (2i, 2i + 1) instead of (i, i + dim / 2).
 "distance_slopes": no rotation; the score of a query with a key loses slope_h x their distance, slope_h =
 2^(-``exponent`` (h + 1) / heads) for head h (``exponent`` 8 unless given).  ``dim``, ``theta``: a rotation besides.
 "none": no position encoding.
@@ -54,7 +56,14 @@ class ScaledRotary(PositionEncoding):
         i = torch.arange(self.dim // 2, dtype=torch.float64)
         freq = self.theta ** (-2.0 * i / self.dim)
         magnitude = 1.0
-        if scaling:
+        if scaling and scaling.get("kind") == "wavelength":
+            factor, original = float(scaling["factor"]), float(scaling["original"])
+            low, high = float(scaling["low"]), float(scaling["high"])
+            turns = original * freq / (2.0 * math.pi)          # turns a pair makes within the original context
+            s = (turns - low) / (high - low)
+            freq = torch.where(turns > high, freq,
+                               torch.where(turns < low, freq / factor, (1.0 - s) * freq / factor + s * freq))
+        elif scaling:
             factor, original = float(scaling["factor"]), float(scaling["original"])
 
             def dim_of(turns: float) -> float:

@@ -33,6 +33,16 @@ output projection.  The slot also carries what the next portion needs of the tok
   q and k rotated by the position encoding (k then times dk^(-1/2)); the read-out is divided by its root mean
   square per head (no gain), times silu(W_g x).  Nothing but S is carried.
 
+"gated_delta" with ``decay`` "head": one decay per head, g = exp(-exp(A_log) softplus(W_a x + dt_bias)), instead of one
+per key channel; with ``gate`` "silu": the gate is silu(W_g x), a whole projection, instead of the low-rank sigmoid.
+
+"mlstm" (per head, the matrix memory of xLSTM, with exponential gates):
+    m_t = max(f_t + m_(t-1), i_t);  S <- e^(f_t + m_(t-1) - m_t) S + e^(i_t - m_t) k_t v_t^T, n <- likewise with k_t alone;
+    o_t = S^T q_t / (max(|n . q_t|, e^(-m_t)) + 1e-6)
+  i = cap tanh((W_i x + b_i) / cap), f = logsigmoid(cap tanh((W_f x + b_f) / cap)), m from 0; q scaled by dk^(-1/2);
+  the read-out is divided by its root mean square per head, times a gain over all heads, times sigmoid(W_g x).  S, n and
+  m are carried.
+
 The projections run as the engine's products (tensor cores in bfloat16); everything between
 them and the recurrence, the recurrence and the state are float32 (csrc/recurrent.cu).
 """
@@ -63,16 +73,40 @@ def _f32(t: torch.Tensor) -> torch.Tensor:
     return t.to(torch.float32).contiguous()
 
 
+def _joined(parts: dict) -> tuple[torch.Tensor, dict]:
+    """One matrix for products of the same rows, each part from a row that is a multiple of 8 (so that kernels and products
+    can take its columns of the result where they lie): (matrix, first row of every part)."""
+    rows, at, row = [], {}, 0
+    for name, w in parts.items():
+        at[name] = row
+        pad = -w.shape[0] % 8
+        rows += [w, torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device)]
+        row += w.shape[0] + pad
+    return torch.cat(rows, dim=0).contiguous(), at
+
+
+def _product(x, w, out, err) -> None:
+    """out = x @ w.T, the norm of ``x`` made inside where it is still to be made and the kernel can."""
+    if isinstance(x, NormedRows):
+        x.linear(w, out, K.EPILOGUE_STORE, err)
+    else:
+        K.gemm_nt(x, w, out, err=err)
+
+
 class GatedDelta(Mixer):
     graph_safe = True
     accepts_normed_rows = True       # its one product of the mixer's input can make the norm itself
 
     def __init__(self, hidden_size, num_heads, num_kv_heads, key_dim, value_dim, conv_taps, norm_eps, unit_eps,
-                 runtime: Runtime, decay_rank=None, gate_rank=None):
+                 runtime: Runtime, decay_rank=None, gate_rank=None, decay="channel", gate="low_rank"):
+        if (decay, gate) not in (("channel", "low_rank"), ("head", "silu")):
+            raise ValueError(f"gated_delta: decay {decay!r} with gate {gate!r} is not supported (channel with low_rank, "
+                             "head with silu)")
+        self.per_head = decay == "head"
         if num_heads % num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
-        if not 1 <= conv_taps <= 8:
-            raise ValueError(f"a convolution of {conv_taps} taps is not supported (1 to 8)")
+        if not 1 <= conv_taps <= 16:
+            raise ValueError(f"a convolution of {conv_taps} taps is not supported (1 to 16)")
         if key_dim > 256:
             raise ValueError(f"key_dim {key_dim} is not supported (up to 256)")
         self.w, self.H, self.G = int(hidden_size), int(num_heads), int(num_kv_heads)
@@ -89,12 +123,18 @@ class GatedDelta(Mixer):
 
     def weight_specs(self):
         taps = ("normal", 0.0, 0.5)
-        return {
+        specs = {
             "q": WeightSpec((self.Kd, self.w)), "k": WeightSpec((self.Kd, self.w)), "v": WeightSpec((self.Vd, self.w)),
             "q.conv": WeightSpec((self.Kd, self.taps), "gain", taps), "k.conv": WeightSpec((self.Kd, self.taps), "gain", taps),
             "v.conv": WeightSpec((self.Vd, self.taps), "gain", taps),
             "b": WeightSpec((self.H, self.w)), "A_log": WeightSpec((self.H,), "gain", ("normal", -1.0, 0.5)),
             "norm": WeightSpec((self.dv,), "gain"),
+        }
+        if self.per_head:
+            return {**specs, "a": WeightSpec((self.H, self.w)), "dt_bias": WeightSpec((self.H,), "gain", ("normal", -1.0, 1.0)),
+                    "g": WeightSpec((self.Vd, self.w)), "o": WeightSpec((self.w, self.Vd))}
+        return {
+            **specs,
             "a1": WeightSpec((self.rank_a, self.w)), "a2": WeightSpec((self.H * self.dk, self.rank_a)),
             "dt_bias": WeightSpec((self.H * self.dk,), "gain", ("normal", -1.0, 1.0)),
             "g1": WeightSpec((self.rank_g, self.w)), "g2": WeightSpec((self.Vd, self.rank_g)),
@@ -102,6 +142,13 @@ class GatedDelta(Mixer):
         }
 
     def bind(self, t):
+        self.conv_w = _f32(torch.cat([t["q.conv"], t["k.conv"], t["v.conv"]], dim=0))
+        self.w_o, self.dt_bias, self.a_log, self.gain = t["o"], _f32(t["dt_bias"]), _f32(t["A_log"]), _f32(t["norm"])
+        if self.per_head:
+            # one product for q, k, v and the gate, and one with a float32 result for beta's and the decay's logits
+            self.w_in, self.at = _joined({"qkv": torch.cat([t["q"], t["k"], t["v"]], dim=0), "g": t["g"]})
+            self.w_gates = torch.cat([t["b"], t["a"]], dim=0).contiguous()
+            return
         if t["a1"].shape[0] != t["a2"].shape[1] or t["g1"].shape[0] != t["g2"].shape[1]:
             raise ValueError("the two halves of a low-rank map do not have the same rank")
         # one product for everything that reads the mixer's input: q, k, v, beta, then (from a column
@@ -113,11 +160,30 @@ class GatedDelta(Mixer):
         self.ra, self.rg = t["a1"].shape[0], t["g1"].shape[0]
         parts.append(zeros(-(self.low_at + self.ra + self.rg) % 8))
         self.w_in = torch.cat(parts, dim=0).contiguous()
-        self.conv_w = _f32(torch.cat([t["q.conv"], t["k.conv"], t["v.conv"]], dim=0))
-        self.w_a2, self.w_g2, self.w_o = t["a2"].contiguous(), t["g2"].contiguous(), t["o"]
-        self.dt_bias, self.a_log, self.gain = _f32(t["dt_bias"]), _f32(t["A_log"]), _f32(t["norm"])
+        self.w_a2, self.w_g2 = t["a2"].contiguous(), t["g2"].contiguous()
+
+    def _forward_per_head(self, x, ctx, cache, residual):
+        rt, tokens = self.rt, residual.shape[0]
+        f32 = torch.float32
+        proj, gates = rt.rows(tokens, self.w_in.shape[0]), rt.rows(tokens, 2 * self.H, dtype=f32)
+        _product(x, self.w_in, proj, rt.err)
+        _product(x, self.w_gates, gates, rt.err)
+        qkv = rt.rows(tokens, self.C, dtype=f32)
+        decay, beta = rt.rows(tokens, self.H, dtype=f32), rt.rows(tokens, self.H, dtype=f32)
+        K.delta_prep(proj, self.conv_w, self.dt_bias, self.a_log, cache.state, ctx.token_slot, qkv, decay, beta,
+                     self.H, self.G, self.dk, self.dv, self.taps, self.unit_eps, gates=gates)
+        portions, cap = portion_list(ctx, cache.state, rt)
+        o = rt.rows(tokens, self.Vd, dtype=f32)
+        K.state_rule(K.RULE_DELTA_HEAD, rt.dtype, portions, cap, cache.state, qkv, None, None, decay, beta, None, o,
+                     proj, self.C, self.taps - 1, self.H, self.G, self.dk, self.dv)
+        y = rt.rows(tokens, self.Vd)
+        at = self.at["g"]
+        K.head_rms_gate(o, self.gain, None, proj[:, at:at + self.Vd], y, self.H, self.dv, True, self.eps)
+        K.gemm_nt(y, self.w_o, residual, K.EPILOGUE_RESIDUAL, err=rt.err)
 
     def forward(self, x, ctx, cache, residual):
+        if self.per_head:
+            return self._forward_per_head(x, ctx, cache, residual)
         rt, tokens = self.rt, residual.shape[0]
         f32 = torch.float32
         proj = rt.rows(tokens, self.w_in.shape[0])
@@ -386,6 +452,65 @@ class Retention(Mixer):
         K.gemm_nt(y, self.w_o, residual, K.EPILOGUE_STORE if overwrite else K.EPILOGUE_RESIDUAL, err=rt.err)
 
 
+class MLstm(Mixer):
+    graph_safe = True
+    accepts_normed_rows = True
+    can_overwrite = True
+
+    def __init__(self, hidden_size, num_heads, key_dim, value_dim, gate_cap, norm_eps, runtime: Runtime, names=None):
+        if key_dim > 512:
+            raise ValueError(f"key_dim {key_dim} is not supported (up to 512)")
+        if not float(gate_cap) > 0:
+            raise ValueError("gate_cap must be positive")
+        self.w, self.H, self.dk, self.dv = int(hidden_size), int(num_heads), int(key_dim), int(value_dim)
+        self.cap, self.eps, self.rt = float(gate_cap), float(norm_eps), runtime
+        self.Kd, self.Vd = self.H * self.dk, self.H * self.dv
+        self.names = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "norm": "norm", "i": "i", "i_bias": "i.b",
+                      "f": "f", "f_bias": "f.b"}
+        self.names.update(names or {})
+
+    def cache_need(self):
+        # S with n as one more column, and m as one more row (csrc/recurrent.cu)
+        return CacheNeed("state", state_shape=(self.H * (self.dk + 1) * (self.dv + 1),), state_dtype=torch.float32)
+
+    def weight_specs(self):
+        n = self.names
+        return {n["q"]: WeightSpec((self.Kd, self.w)), n["k"]: WeightSpec((self.Kd, self.w)), n["v"]: WeightSpec((self.Vd, self.w)),
+                n["g"]: WeightSpec((self.Vd, self.w)), n["o"]: WeightSpec((self.w, self.Vd)), n["norm"]: WeightSpec((self.Vd,), "gain"),
+                n["i"]: WeightSpec((self.H, self.w)), n["i_bias"]: WeightSpec((self.H,), "gain", ("normal", 0.0, 1.0)),
+                n["f"]: WeightSpec((self.H, self.w)), n["f_bias"]: WeightSpec((self.H,), "gain", ("normal", 3.0, 1.0))}
+
+    def bind(self, t):
+        n = self.names
+        self.w_in, self.at = _joined({s: t[n[s]] for s in ("q", "k", "v", "g")})
+        # the gates' logits are a product of their own, with a float32 result
+        self.w_gates = torch.cat([t[n["i"]], t[n["f"]]], dim=0).contiguous()
+        self.gate_bias = _f32(torch.cat([t[n["i_bias"]], t[n["f_bias"]]]))
+        self.gain, self.w_o = _f32(t[n["norm"]]), t[n["o"]]
+
+    def forward(self, x, ctx, cache, residual, overwrite=False):
+        rt, tokens, at = self.rt, residual.shape[0], self.at
+        proj, gates = rt.rows(tokens, self.w_in.shape[0]), rt.rows(tokens, 2 * self.H, dtype=torch.float32)
+        _product(x, self.w_in, proj, rt.err)
+        _product(x, self.w_gates, gates, rt.err)
+        portions, cap = portion_list(ctx, cache.state, rt)
+        o = rt.rows(tokens, self.H * (self.dv + 2), dtype=torch.float32)
+        K.state_rule(K.RULE_MLSTM, rt.dtype, portions, cap, cache.state, proj[:, at["q"]:at["q"] + self.Kd],
+                     proj[:, at["k"]:at["k"] + self.Kd], proj[:, at["v"]:at["v"] + self.Vd], gates, None, None, o,
+                     None, 0, 0, self.H, self.H, self.dk, self.dv, out_scale=self.dk ** -0.5, gate_bias=self.gate_bias,
+                     gate_cap=self.cap)
+        y = rt.rows(tokens, self.Vd)
+        K.head_rms_gate(o, self.gain, None, proj[:, at["g"]:at["g"] + self.Vd], y, self.H, self.dv, False, self.eps,
+                        gate_logit=True, normalized=True)
+        K.gemm_nt(y, self.w_o, residual, K.EPILOGUE_STORE if overwrite else K.EPILOGUE_RESIDUAL, err=rt.err)
+
+
+@register_part("mixer", "mlstm")
+def _build_mlstm(spec, runtime, **_):
+    return MLstm(spec["hidden_size"], spec["num_heads"], spec["key_dim"], spec["value_dim"], spec["gate_cap"],
+                 spec["norm_eps"], runtime, names=spec.get("names"))
+
+
 @register_part("mixer", "gated_recurrent_unit")
 def _build_unit(spec, runtime, **_):
     return GatedRecurrentUnit(spec["hidden_size"], spec["width"], spec["blocks"], spec["conv_taps"], runtime,
@@ -408,7 +533,8 @@ def _build_gated_linear(spec, runtime, **_):
 def _build_delta(spec, runtime, **_):
     return GatedDelta(spec["hidden_size"], spec["num_heads"], spec["num_kv_heads"], spec["key_dim"],
                       spec["value_dim"], spec["conv_taps"], spec["norm_eps"], spec.get("unit_eps", 1e-6), runtime,
-                      decay_rank=spec.get("decay_rank"), gate_rank=spec.get("gate_rank"))
+                      decay_rank=spec.get("decay_rank"), gate_rank=spec.get("gate_rank"),
+                      decay=spec.get("decay", "channel"), gate=spec.get("gate", "low_rank"))
 
 
 @register_part("mixer", "wkv")
