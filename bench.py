@@ -38,6 +38,7 @@ bias beside gated linear attention, attention over a cached latent, a clamped ga
 two of the layers run twice) beside Qwen3 layers of equal width, depth, head counts and
 feed-forward size.
 ``--workload pikurax`` does the same for the Pikurax design beside Malazen.
+``--workload kusolorn`` does the same for the Kusolorn design beside Sevipel and Malazen.
 ``--workload kemirax`` does the same for the Kemirax design (one norm feeding a mixer behind a token
 shift and routed experts side by side, gates on both; attention over a cached latent with queries
 through a latent and layers that read another layer's cache; gated linear attention; identity and
@@ -576,7 +577,8 @@ def kernel_times(runner, entries_of, steps=3):
              "tanh_rows", "double_exp_decay", "state_rule", "head_rms_gate", "experts_route", "experts_plan", "experts_product",
              "experts_product_tc", "experts_gather", "experts_combine", "latent_finish", "heads_product",
              "sigmoid_power_decay", "clamped_glu", "row_bias", "weighted_sum", "gated_sum", "experts_mix", "rmsnorm_shift", "experts_route_plan",
-             "layernorm", "norm_merge_add", "pair_embed", "rows_cast", "scale_cap", "unit_gates", "unit_scan", "rotate_rows"]
+             "layernorm", "norm_merge_add", "pair_embed", "rows_cast", "scale_cap", "unit_gates", "unit_scan", "rotate_rows",
+             "side_gate"]
     records, saved, graphs, turn = [], {}, runner.graphs, [0]
     runner.graphs = None
 
@@ -584,7 +586,8 @@ def kernel_times(runner, entries_of, steps=3):
         def timed(*a, **kw):
             label = name
             if name == "state_rule":
-                label = {K.RULE_DELTA: "delta_rule", K.RULE_WKV: "wkv_rule", K.RULE_GLA: "gla_rule"}[a[0]]
+                label = {K.RULE_DELTA: "delta_rule", K.RULE_WKV: "wkv_rule", K.RULE_GLA: "gla_rule",
+                         K.RULE_DELTA_HEAD: "delta_head_rule", K.RULE_MLSTM: "mlstm_rule"}[a[0]]
             elif name in ("experts_product", "experts_product_tc"):
                 # (a feed-forward of experts makes its first product, then its second)
                 turn[0] ^= 1
@@ -1096,6 +1099,129 @@ def run_pikurax(args):
     return 0
 
 
+KUSOLORN_SIZES = {
+    "w1024": {"width": 1024, "heads": 8, "kv_heads": 4, "linear_heads": 4, "experts": 16, "top": 2, "expert_ff": 768, "ff": 4096,
+              "side": 128, "window": 1024},
+    "w2048": {"width": 2048, "heads": 16, "kv_heads": 4, "linear_heads": 8, "experts": 32, "top": 4, "expert_ff": 768,
+              "ff": 8192, "side": 256, "window": 1024},
+}
+KUSOLORN_KEPT = 4
+
+
+def kusolorn_config(z):
+    """Eight layers: three with an mLSTM (Malazen's linear heads of this file), three with the gated delta rule and two with
+    attention (Sevipel's heads, experts and window of this file; the first four positions stay visible, scores capped); four
+    have a dense feed-forward, four experts; every layer takes a row of the token's own."""
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0}, "router": {"experts": z["experts"], "top": z["top"]}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+           "v_mix": True, "mask": {"size": z["window"], "keep_first": KUSOLORN_KEPT},
+           "rot": {"dims": 64, "base": 1000000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 1024}}}
+    delta = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": 128, "vdim": 128, "conv": 4}
+    lstm = {"heads": z["linear_heads"], "dim": 128, "vdim": 128, "gate_cap": 15.0}
+    kinds = [("mlstm", lstm, dense), ("delta", delta, moe), ("attention", att, dense), ("mlstm", lstm, moe),
+             ("delta", delta, dense), ("attention", att, moe), ("mlstm", lstm, dense), ("delta", delta, moe)]
+    return {"architecture": "Kusolorn", "vocab": DESIGN_VOCAB, "width": z["width"], "norm": {"eps": 1e-5}, "max_positions": 4096,
+            "token_side": {"dim": z["side"]},
+            "layers": [{"type": t, "mixer": json.loads(json.dumps(m)), "mlp": json.loads(json.dumps(f))} for t, m, f in kinds]}
+
+
+def run_kusolorn(args):
+    pk = peaks()
+    tokens, batch, context = PREFILL_TOKENS, 8, DESIGN_CONTEXT
+    sizes = {}
+    clocks = ClockSampler()
+    clocks.start()
+    for size, z in KUSOLORN_SIZES.items():
+        sz, mz = DESIGN_SIZES[size], MALAZEN_SIZES[size]
+        row = {"kusolorn": measure_design(kusolorn_config(z), args, tokens, batch, context),
+               "sevipel": measure_design(design_configs(sz)[0], args, tokens, batch, context),
+               "malazen": measure_design(malazen_configs(mz)[0], args, tokens, batch, context)}
+        w, H, G, LH, ff, side = z["width"], z["heads"], z["kv_heads"], z["linear_heads"], z["ff"], z["side"]
+        n_lstm, n_delta, n_att, n_dense, n_moe = 3, 3, 2, 4, 4
+        # products of a prefill through the engine's product kernels (the experts' apart)
+        lstm_cols = 4 * LH * 128 + 2 * LH + LH * 128
+        delta_cols = 2 * G * 128 + 2 * H * 128 + 2 * H + H * 128
+        att_cols = (H + 2 * G) * 128 + H * 128
+        flops_k = 2 * tokens * w * (n_lstm * lstm_cols + n_delta * delta_cols + n_att * att_cols + n_dense * 2 * ff
+                                    + n_moe * z["experts"] + 8 * 2 * side) + 2 * DESIGN_VOCAB * w
+        rank = sz["rank"]
+        s_delta = (2 * G * 128 + H * 128 + H + 2 * rank) * w + rank * 2 * H * 128 + H * 128 * w
+        s_wkv = 5 * sz["wkv_heads"] * 64 * w + rank * (w + sz["wkv_heads"] * 64)
+        flops_s = 2 * tokens * (4 * s_delta + 2 * s_wkv + (2 * H + 2 * G + 2 * H) * 128 * w + 8 * sz["experts"] * w) \
+            + 2 * DESIGN_VOCAB * w
+        MLH, MQH, mff = mz["linear_heads"], mz["latent_heads"], mz["ff"]
+        R, DR, DP, DV = MALAZEN_RANK, MALAZEN_ROT, MALAZEN_PLAIN, MALAZEN_VALUE
+        par_cols = (mz["heads"] + 2 * mz["kv_heads"]) * 128 + mz["heads"] * 128 + 5 * MLH * 128 + 64
+        flops_m = 2 * tokens * w * (3 * par_cols + 5 * (MQH * (DP + DR) + R + DR + MQH * DV) + 8 * 3 * mff) + 2 * DESIGN_VOCAB * w
+        pairs_win = sum(min(i + 1, z["window"]) for i in range(tokens))
+        pairs_kept = sum(min(max(i + 1 - z["window"], 0), KUSOLORN_KEPT) for i in range(tokens))
+        att_k, att_s = n_att * 4 * (pairs_win + pairs_kept) * H * 128, 2 * 4 * pairs_win * H * 128
+        experts_k, experts_s = 2 * tokens * z["top"] * z["expert_ff"] * w * n_moe, 2 * tokens * sz["top"] * sz["ff"] * w * 8
+        cache_k = 2 * batch * n_att * (z["window"] + KUSOLORN_KEPT) * 2 * G * 128
+        cache_s = 2 * batch * 2 * sz["window"] * 2 * G * 128
+        state = lambda heads, layers: 2 * 4 * batch * layers * heads * 128 * 128
+        stream = 4 * tokens * w                     # one float32 pass over the step's rows
+
+        def frac(amount, ms, peak):
+            return round(amount / (ms * 1e-3) / peak, 4) if ms else None
+
+        def ms_of(kernels, *names):
+            return sum(kernels.get(n, 0.0) for n in names)
+
+        tf, bw = pk["bf16_tflops"] * 1e12, pk["hbm_gbs"] * 1e9
+        products = ("gemm_nt_tc", "gemm_nt_tc_rmsnorm")
+        attention = ("attention_tile", "attention_prefill_tc")
+        decode_attention = ("attention_decode", "attention_decode_mma", "attention_tile")
+        kp, sp, mp = (row[d]["prefill_kernels_ms"] for d in ("kusolorn", "sevipel", "malazen"))
+        kd, sd, md = (row[d]["decode_kernels_ms"] for d in ("kusolorn", "sevipel", "malazen"))
+        per_token = lambda kernels, name, layers: round(ms_of(kernels, name) * 1e3 / (layers * tokens), 4)
+        row["like_kernels_fraction_of_measured_peak [kusolorn, like kernel]"] = {
+            "prefill: products (tensor cores); sevipel, malazen": [frac(flops_k, ms_of(kp, *products), tf),
+                                                                   frac(flops_s, ms_of(sp, *products), tf),
+                                                                   frac(flops_m, ms_of(mp, *products), tf)],
+            "prefill: attention in a window; sevipel": [frac(att_k, ms_of(kp, *attention), tf), frac(att_s, ms_of(sp, *attention), tf)],
+            "prefill: delta rule, microseconds a token and layer; sevipel": [per_token(kp, "delta_head_rule", n_delta),
+                                                                             per_token(sp, "delta_rule", 4)],
+            "prefill: what comes before the delta rule (delta_prep), bytes; sevipel": [
+                frac(n_delta * tokens * ((2 * G + H) * 128 * 6 + H * 16), ms_of(kp, "delta_prep"), bw),
+                frac(4 * tokens * ((2 * G + H) * 128 * 6 + H * 128 * 8), ms_of(sp, "delta_prep"), bw)],
+            "prefill: mlstm rule, microseconds a token and layer; malazen's gated linear rule": [
+                per_token(kp, "mlstm_rule", n_lstm), per_token(mp, "gla_rule", 3)],
+            "prefill: experts' first product; sevipel": [frac(2 * experts_k, ms_of(kp, "experts_up"), tf),
+                                                         frac(experts_s, ms_of(sp, "experts_up"), tf)],
+            "prefill: experts' second product; sevipel": [frac(experts_k, ms_of(kp, "experts_down"), tf),
+                                                          frac(experts_s, ms_of(sp, "experts_down"), tf)],
+            "prefill: clamped gated activation (bytes read and written); malazen": [
+                frac(n_moe * tokens * z["top"] * z["expert_ff"] * 10, ms_of(kp, "clamped_glu"), bw),
+                frac(8 * tokens * mff * 10, ms_of(mp, "clamped_glu"), bw)],
+            "prefill: q, k, v finished (qkv_finish), bytes; sevipel": [
+                frac(n_att * tokens * (H + 2 * G) * 128 * 4, ms_of(kp, "qkv_finish"), bw),
+                frac(2 * tokens * (H + G) * 128 * 4, ms_of(sp, "qkv_finish"), bw)],
+            "prefill: read-out's norm and gate (head_rms_gate), bytes; sevipel": [
+                frac(tokens * 8 * 128 * (n_lstm * LH + n_delta * H), ms_of(kp, "head_rms_gate"), bw),
+                frac(tokens * (4 * 10 * 128 * H + 2 * 8 * 64 * sz["wkv_heads"]), ms_of(sp, "head_rms_gate"), bw)],
+            "prefill: the token input's closing kernel (3 passes); malazen's weighted_sum (4)": [
+                frac(8 * 3 * stream, ms_of(kp, "norm_merge_add", "side_close"), bw), frac(3 * 4 * stream, ms_of(mp, "weighted_sum"), bw)],
+            "prefill: norm in front of a sublayer; sevipel": [frac(16 * tokens * w * 6, ms_of(kp, "rmsnorm"), bw),
+                                                              frac(16 * tokens * w * 6, ms_of(sp, "rmsnorm"), bw)],
+            "decode: attention (bytes of cache); sevipel": [frac(cache_k, ms_of(kd, *decode_attention), bw),
+                                                            frac(cache_s, ms_of(sd, *decode_attention), bw)],
+            "decode: delta rule (bytes of state); sevipel": [frac(state(H, n_delta), ms_of(kd, "delta_head_rule"), bw),
+                                                             frac(state(H, 4), ms_of(sd, "delta_rule"), bw)],
+            "decode: mlstm rule (bytes of state); malazen": [frac(state(LH, n_lstm), ms_of(kd, "mlstm_rule"), bw),
+                                                             frac(state(MLH, 3), ms_of(md, "gla_rule"), bw)],
+        }
+        sizes[size] = row
+    clock = clocks.stop()
+    print(json.dumps({
+        "metric": "prefill of 2,048 tokens and decode at batch 8, context 2,048: Kusolorn beside Sevipel and Malazen at equal size",
+        "unit": "ms, tok/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic", "impl": "ours", "clocks": clock,
+        "peaks": pk, "layer_runs": 8, "vocab": DESIGN_VOCAB, "sizes": sizes,
+    }))
+    return 0
+
+
 # ---------------------------------------------------------------------------
 # the reference arm: LockStep itself, unmodified, from baseline/_ref
 # ---------------------------------------------------------------------------
@@ -1265,9 +1391,9 @@ def main():
     ap.add_argument("--no-fp32", action="store_true", help="skip the float32 points")
     ap.add_argument("--only", default="", choices=["", "decode", "prefill"],
                     help="time only this part and print a short line (for profiling a small case)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "designs", "malazen", "kemirax", "pikurax"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "designs", "malazen", "kemirax", "pikurax", "kusolorn"],
                     help="mixed: a continuous batch of 64 requests through the entry point; designs: the Sevipel "
-                         "design beside Qwen3 layers of equal size, with every kernel's time; malazen, kemirax, pikurax: the same "
+                         "design beside Qwen3 layers of equal size, with every kernel's time; malazen, kemirax, pikurax, kusolorn: the same "
                          "for those designs")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
                     help="element type of the --only runs (the full line always reports both)")
@@ -1292,6 +1418,8 @@ def main():
         return run_kemirax(args)
     if args.workload == "pikurax":
         return run_pikurax(args)
+    if args.workload == "kusolorn":
+        return run_kusolorn(args)
     return run_ours(args)
 
 

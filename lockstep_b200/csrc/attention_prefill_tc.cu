@@ -109,11 +109,10 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
-// tanh x on the special-function unit, one instruction
-__device__ __forceinline__ float tanh_approx(float x) {
-  float y;
-  asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
+// tanh x = 1 - 2 / (1 + e^(2 x)), to float32 accuracy relative to one: what a capped score needs, which is this times the
+// cap (the one-instruction tanh of the special-function unit keeps eleven bits)
+__device__ __forceinline__ float tanh_of(float x) {
+  return 1.0f - __fdividef(2.0f, 1.0f + ex2(x * 2.8853900817779268f));
 }
 
 // lg2 x on the special-function unit, one instruction (inputs here are >= 1)
@@ -173,7 +172,7 @@ struct Item {
 // slopes[head] x lg2(1 + log_rates[head] x distance), one more special-function instruction a score),
 // and the softmax's denominator one more term exp(sinks[head]) at the end of a row.  With slopes and no log_rates the
 // bias is slopes[head] x distance, and with cap_log2 > 0 (a cap times lg2 e) the scaled score first becomes
-// cap tanh(score / cap): one tanh.approx a score, again in the units of the exponentials.  keep_first > 0: the first
+// cap tanh(score / cap), again in the units of the exponentials.  keep_first > 0: the first
 // keep_first keys of the sequence stay visible behind the window; their tiles come first.
 template <int HALVES, bool EXTRAS>
 __global__ void __launch_bounds__(THREADS, 1)
@@ -476,7 +475,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             for (int jj = 0; jj < HC; ++jj) {
               const float dist = fmaxf(d0 - (float)jj, 0.f);
               const float raw = __uint_as_float(sc[jj]);
-              const float v = capped ? cap_log2 * tanh_approx(raw * bias_b) : raw * scale_log2;
+              const float v = capped ? cap_log2 * tanh_of(raw * bias_b) : raw * scale_log2;
               sc[jj] = __float_as_uint(fmaf(-bias_a, dist, v));
             }
           } else if (biased) {
