@@ -124,7 +124,7 @@ _SIGNATURES["seq"] = {
     "ls_double_exp_decay": [c_void_p, c_void_p, ctypes.c_longlong, c_int, c_void_p],
     "ls_shift_mix": [c_void_p, c_int, c_void_p, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_int, c_int, c_int,
                      c_void_p],
-    "ls_state_rule": [c_int, c_int, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
+    "ls_state_rule": [c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
                       c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
                       c_int64, c_float, c_int64, c_void_p, c_float, c_void_p],
     "ls_unit_gates": [c_void_p, ctypes.c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong,
@@ -966,7 +966,7 @@ def state_rule(rule: int, dtype, portions, max_portions: int, state, in_a, in_b,
     else:
         pa, pb, pv = _dev(in_a, "in_a"), _opt(in_b, "in_b"), _opt(in_v, "in_v")
     _check(library("seq").ls_state_rule(
-        rule, _DTYPE_CODE[dtype], _dev(portions, "portions", torch.int32), max_portions,
+        rule, _DTYPE_CODE[dtype], _dev(portions, "portions", torch.int32), max_portions, out.shape[0],
         _dev(state, "state", torch.float32), state.shape[1], pa, pb, pv,
         _dev(decay, "decay", torch.float32), _opt(beta, "beta", torch.float32), _opt(bonus, "bonus", torch.float32),
         _dev(out, "out", torch.float32), _opt(carry_src, "carry_src", dtype),
