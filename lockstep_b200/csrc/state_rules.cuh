@@ -140,9 +140,99 @@ __device__ __forceinline__ void fold_lanes(float (&o)[UNIT], int part) {
 }
 __host__ __device__ constexpr int log2_of(int n) { return n <= 1 ? 0 : 1 + log2_of(n / 2); }
 
-// SHORT: for steps of single tokens: the walk token by token only, with fewer registers, so that more blocks run at a time.
-template <int RULE, int L, bool SHORT>
-__global__ void __launch_bounds__(STAGERS + 32 * MAX_WALK_WARPS + (RULE == RULE_MLSTM ? 32 : 0), SHORT ? 2 : 1)
+// This thread's channels of what a token brings.
+struct TokenRows {
+  ulonglong2 a[ROWS / 4], b[ROWS / 4], d[ROWS / 4];      // queries, keys, decays
+};
+
+// One token: the state's update, and this thread's share of the read-out.  `v`: the column's value; `beta`: of a delta
+// rule; `keep`: the one decay of a rule that has one.
+template <int RULE, int L>
+__device__ __forceinline__ float advance(f32x2 (&S)[ROWS / 2], const f32x2* bonus, const TokenRows& t, float v, float beta,
+                                         float keep) {
+  constexpr bool DELTA = RULE == RULE_DELTA || RULE == RULE_DELTA_HEAD;
+  constexpr bool ONE_DECAY = RULE == RULE_DELTA_HEAD || RULE == RULE_MLSTM;
+  const f32x2 one_decay = pack2(keep, keep);
+  f32x2 o01 = 0ull, o23 = 0ull;
+  if constexpr (DELTA) {
+    f32x2 d01 = 0ull, d23 = 0ull;
+#pragma unroll
+    for (int r = 0; r < ROWS / 4; ++r) {
+      S[2 * r] = mul2(S[2 * r], ONE_DECAY ? one_decay : t.d[r].x); d01 = fma2(S[2 * r], t.b[r].x, d01);
+      S[2 * r + 1] = mul2(S[2 * r + 1], ONE_DECAY ? one_decay : t.d[r].y); d23 = fma2(S[2 * r + 1], t.b[r].y, d23);
+    }
+    float dot = sum_chains(d01, d23);
+#pragma unroll
+    for (int off = L >> 1; off > 0; off >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, off);
+    const float u = beta * (v - dot);
+    const f32x2 u2 = pack2(u, u);
+#pragma unroll
+    for (int r = 0; r < ROWS / 4; ++r) {
+      S[2 * r] = fma2(t.b[r].x, u2, S[2 * r]); o01 = fma2(S[2 * r], t.a[r].x, o01);
+      S[2 * r + 1] = fma2(t.b[r].y, u2, S[2 * r + 1]); o23 = fma2(S[2 * r + 1], t.a[r].y, o23);
+    }
+  } else {
+    const f32x2 v2 = pack2(v, v);
+#pragma unroll
+    for (int r = 0; r < ROWS / 4; ++r) {
+      const f32x2 kx = mul2(t.b[r].x, v2), ky = mul2(t.b[r].y, v2);
+      const f32x2 dx = ONE_DECAY ? one_decay : t.d[r].x, dy = ONE_DECAY ? one_decay : t.d[r].y;
+      if constexpr (RULE == RULE_WKV) {
+        o01 = fma2(t.a[r].x, fma2(bonus[2 * r], kx, S[2 * r]), o01); S[2 * r] = fma2(dx, S[2 * r], kx);
+        o23 = fma2(t.a[r].y, fma2(bonus[2 * r + 1], ky, S[2 * r + 1]), o23); S[2 * r + 1] = fma2(dy, S[2 * r + 1], ky);
+      } else {
+        S[2 * r] = fma2(dx, S[2 * r], kx); o01 = fma2(t.a[r].x, S[2 * r], o01);
+        S[2 * r + 1] = fma2(dy, S[2 * r + 1], ky); o23 = fma2(t.a[r].y, S[2 * r + 1], o23);
+      }
+    }
+  }
+  return sum_chains(o01, o23);
+}
+
+// The logs of an mlstm's input and forget gates from their logits.
+__device__ __forceinline__ float log_input_gate(float z, float bias, float cap) { return cap * tanhf((z + bias) / cap); }
+__device__ __forceinline__ float log_forget_gate(float z, float bias, float cap) {
+  return -softplus_f(-cap * tanhf((z + bias) / cap));
+}
+
+// The state of this thread's column, its channels part * ROWS ..., between memory and register pairs.
+__device__ __forceinline__ void load_state(const float* state, int cols, int col, bool active, int part, int dk,
+                                           f32x2 (&S)[ROWS / 2]) {
+#pragma unroll
+  for (int r = 0; r < ROWS / 2; ++r) {
+    const int i = part * ROWS + 2 * r;
+    S[r] = pack2((active && i < dk) ? state[(int64_t)i * cols + col] : 0.f,
+                 (active && i + 1 < dk) ? state[(int64_t)(i + 1) * cols + col] : 0.f);
+  }
+}
+__device__ __forceinline__ void store_state(float* state, int cols, int col, int part, int dk, const f32x2 (&S)[ROWS / 2]) {
+#pragma unroll
+  for (int r = 0; r < ROWS / 2; ++r) {
+    const int i = part * ROWS + 2 * r;
+    float x, y;
+    unpack2(S[r], x, y);
+    if (i < dk) state[(int64_t)i * cols + col] = x;
+    if (i + 1 < dk) state[(int64_t)(i + 1) * cols + col] = y;
+  }
+}
+
+// The rest of the state: the last inputs of a portion (its first token t0, n tokens), behind those that were carried.
+__device__ __forceinline__ void carry_inputs(const RuleArgs& a, int slot, int t0, int n) {
+  float* carried = a.state + (int64_t)slot * a.state_stride + (int64_t)a.H * a.dk * a.dv;
+  const int rows = a.carry_rows, W = a.carry_width;
+  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+    float keep[MAX_TAPS];
+    for (int s = 0; s < rows; ++s) {
+      const int from = n - rows + s;
+      keep[s] = from >= 0 ? engine_value(a.carry_src, (int64_t)(t0 + from) * a.carry_ld + c, a.bf16)
+                          : carried[(int64_t)(s + n) * W + c];
+    }
+    for (int s = 0; s < rows; ++s) carried[(int64_t)s * W + c] = keep[s];
+  }
+}
+
+template <int RULE, int L>
+__global__ void __launch_bounds__(STAGERS + 32 * MAX_WALK_WARPS + (RULE == RULE_MLSTM ? 32 : 0), 1)
 rule_kernel(RuleArgs a) {
   extern __shared__ float smem[];
   ls_dependency_sync();
@@ -189,68 +279,26 @@ rule_kernel(RuleArgs a) {
     const int cl = tid / L, part = tid % L, col = col0 + cl;
     const bool active = col < cols;
     // a thread keeps the key channels i = part * ROWS + r of its column, two to a register pair
-    f32x2 S[ROWS / 2], bonus[RULE == RULE_WKV ? ROWS / 2 : 1];
-#pragma unroll
-    for (int r = 0; r < ROWS / 2; ++r) {
-      const int i = part * ROWS + 2 * r;
-      S[r] = pack2((active && i < dk) ? state[(int64_t)i * cols + col] : 0.f,
-                   (active && i + 1 < dk) ? state[(int64_t)(i + 1) * cols + col] : 0.f);
-      if (RULE == RULE_WKV) bonus[r] = pack2(i < dk ? a.bonus[h * dk + i] : 0.f, i + 1 < dk ? a.bonus[h * dk + i + 1] : 0.f);
-    }
+    f32x2 S[ROWS / 2], bonus[ROWS / 2];
+    load_state(state, cols, col, active, part, dk, S);
+    if (RULE == RULE_WKV) load_state(a.bonus + h * dk, 1, 0, true, part, dk, bonus);
     float* out = a.out + ((int64_t)t0 * a.H + h) * out_cols + col;
     const int64_t out_step = (int64_t)a.H * out_cols;
 
-    // one token: the state's update, and this thread's share of the read-out
     auto token = [&](const float* tok, const float4& gate) {
       const ulonglong2* A = reinterpret_cast<const ulonglong2*>(tok + part * run);
       const ulonglong2* B = reinterpret_cast<const ulonglong2*>(tok + dkp + part * run);
       const ulonglong2* D = reinterpret_cast<const ulonglong2*>(tok + 2 * dkp + part * run);
-      const float vj = RULE == RULE_MLSTM ? tok[v_at + cl] * gate.x : tok[v_at + cl];
-      const float keep = RULE == RULE_MLSTM ? gate.y : RULE == RULE_DELTA_HEAD ? tok[n_at + 1] : 0.f;
-      const f32x2 one_decay = pack2(keep, keep);
-      f32x2 o01 = 0ull, o23 = 0ull;
-      if constexpr (DELTA) {
-        f32x2 d01 = 0ull, d23 = 0ull;
-        ulonglong2 kk[ROWS / 4];
+      TokenRows rows_of;
 #pragma unroll
-        for (int r = 0; r < ROWS / 4; ++r) {
-          kk[r] = B[r];
-          ulonglong2 dd;
-          if constexpr (ONE_DECAY) dd.x = dd.y = one_decay;
-          else dd = D[r];
-          S[2 * r] = mul2(S[2 * r], dd.x); d01 = fma2(S[2 * r], kk[r].x, d01);
-          S[2 * r + 1] = mul2(S[2 * r + 1], dd.y); d23 = fma2(S[2 * r + 1], kk[r].y, d23);
-        }
-        float dot = sum_chains(d01, d23);
-#pragma unroll
-        for (int off = L >> 1; off > 0; off >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, off);
-        const float u = tok[n_at] * (vj - dot);
-        const f32x2 u2 = pack2(u, u);
-#pragma unroll
-        for (int r = 0; r < ROWS / 4; ++r) {
-          const ulonglong2 qq = A[r];
-          S[2 * r] = fma2(kk[r].x, u2, S[2 * r]); o01 = fma2(S[2 * r], qq.x, o01);
-          S[2 * r + 1] = fma2(kk[r].y, u2, S[2 * r + 1]); o23 = fma2(S[2 * r + 1], qq.y, o23);
-        }
-      } else {
-        const f32x2 v2 = pack2(vj, vj);
-#pragma unroll
-        for (int r = 0; r < ROWS / 4; ++r) {
-          const ulonglong2 qq = A[r], kk = B[r];
-          ulonglong2 dd;
-          if constexpr (ONE_DECAY) dd.x = dd.y = one_decay;
-          else dd = D[r];
-          const f32x2 kx = mul2(kk.x, v2), ky = mul2(kk.y, v2);
-          if constexpr (COLUMNS) {
-            S[2 * r] = fma2(dd.x, S[2 * r], kx); o01 = fma2(qq.x, S[2 * r], o01);
-            S[2 * r + 1] = fma2(dd.y, S[2 * r + 1], ky); o23 = fma2(qq.y, S[2 * r + 1], o23);
-          } else {
-            o01 = fma2(qq.x, fma2(bonus[2 * r], kx, S[2 * r]), o01); S[2 * r] = fma2(dd.x, S[2 * r], kx);
-            o23 = fma2(qq.y, fma2(bonus[2 * r + 1], ky, S[2 * r + 1]), o23); S[2 * r + 1] = fma2(dd.y, S[2 * r + 1], ky);
-          }
-        }
+      for (int r = 0; r < ROWS / 4; ++r) {
+        rows_of.a[r] = A[r];
+        rows_of.b[r] = B[r];
+        if (!ONE_DECAY) rows_of.d[r] = D[r];
       }
-      return sum_chains(o01, o23);
+      const float v = RULE == RULE_MLSTM ? tok[v_at + cl] * gate.x : tok[v_at + cl];
+      return advance<RULE, L>(S, bonus, rows_of, v, DELTA ? tok[n_at] : 0.f,
+                              RULE == RULE_MLSTM ? gate.y : RULE == RULE_DELTA_HEAD ? tok[n_at + 1] : 0.f);
     };
     auto gate_of = [&](int t) {
       return RULE == RULE_MLSTM ? numbers[t & (2 * GATED - 1)] : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -284,7 +332,7 @@ rule_kernel(RuleArgs a) {
     for (int c = 0; c < chunks; ++c) {
       const float* buf = buffer(c);
       const int c0 = c * CHUNK;
-      if (!SHORT && n - c0 >= CHUNK) {
+      if (n - c0 >= CHUNK) {
 #pragma unroll 1
         for (int u = 0; u < CHUNK; u += UNIT) {
           float o[UNIT];
@@ -308,17 +356,8 @@ rule_kernel(RuleArgs a) {
       }
       meet();
     }
-    if (!SHORT) finish_unit();
-    if (active) {
-#pragma unroll
-      for (int r = 0; r < ROWS / 2; ++r) {
-        const int i = part * ROWS + 2 * r;
-        float x, y;
-        unpack2(S[r], x, y);
-        if (i < dk) state[(int64_t)i * cols + col] = x;
-        if (i + 1 < dk) state[(int64_t)(i + 1) * cols + col] = y;
-      }
-    }
+    finish_unit();
+    if (active) store_state(state, cols, col, part, dk, S);
     if (RULE == RULE_MLSTM) {
       meet();                                        // the running maximum after the last token
       if (active && part == 0) state[(int64_t)dk * cols + col] = numbers[0].x;
@@ -339,8 +378,7 @@ rule_kernel(RuleArgs a) {
     };
     auto make = [&](int round) {
       const int left = n - round * GATED;
-      const float i_mine = cap * tanhf((z_i + bias_i) / cap);
-      const float f_mine = -softplus_f(-cap * tanhf((z_f + bias_f) / cap));
+      const float i_mine = log_input_gate(z_i, bias_i, cap), f_mine = log_forget_gate(z_f, bias_f, cap);
       float keep = 0.f, put = 0.f, floor = 0.f;
 #pragma unroll
       for (int s = 0; s < GATED; ++s) {
@@ -561,34 +599,126 @@ rule_kernel(RuleArgs a) {
     if (RULE == RULE_MLSTM) meet();
   }
 
-  // the rest of the state: the last inputs of this portion, behind those that were carried
-  if (blockIdx.x == 0 && blockIdx.y == 0 && a.carry_rows > 0) {
-    float* carried = a.state + (int64_t)slot * a.state_stride + (int64_t)a.H * dk * dv;
-    const int keep_rows = a.carry_rows, W = a.carry_width;
-    for (int c = tid; c < W; c += blockDim.x) {
-      float keep[MAX_TAPS];
-      for (int s = 0; s < keep_rows; ++s) {
-        const int from = n - keep_rows + s;
-        keep[s] = from >= 0 ? engine_value(a.carry_src, (int64_t)(t0 + from) * a.carry_ld + c, a.bf16)
-                            : carried[(int64_t)(s + n) * W + c];
-      }
-      for (int s = 0; s < keep_rows; ++s) carried[(int64_t)s * W + c] = keep[s];
-    }
-  }
+  if (blockIdx.x == 0 && blockIdx.y == 0 && a.carry_rows > 0) carry_inputs(a, slot, t0, n);
 }
 
-template <int RULE, int L, bool SHORT>
-int launch_as(RuleArgs& a, int max_portions, cudaStream_t stream) {
+// Steps of single tokens: every thread fetches what it needs of a token itself, beside its part of the state (nothing is
+// staged and nobody is waited for).  Portions of several tokens are walked too, each token's fetch in front of it.
+constexpr int STEP_THREADS = 128;
+
+template <int RULE, int L>
+__global__ void __launch_bounds__(STEP_THREADS, 4) rule_step_kernel(RuleArgs a) {
+  ls_dependency_sync();
+  const int p = blockIdx.z;
+  if (p >= a.portions[0]) return;
+  const int t0 = a.portions[1 + 3 * p], n = a.portions[1 + 3 * p + 1], slot = a.portions[1 + 3 * p + 2];
+  constexpr bool DELTA = RULE == RULE_DELTA || RULE == RULE_DELTA_HEAD;
+  constexpr bool ONE_DECAY = RULE == RULE_DELTA_HEAD || RULE == RULE_MLSTM;
+  constexpr bool COLUMNS = RULE == RULE_GLA || RULE == RULE_MLSTM;
+  const int h = blockIdx.y, tid = threadIdx.x, dk = a.dk, dv = a.dv;
+  const int cols = RULE == RULE_MLSTM ? dv + 1 : dv, rows = RULE == RULE_MLSTM ? dk + 1 : dk;
+  const int out_cols = RULE == RULE_MLSTM ? dv + 2 : dv;
+  const int part = tid % L, col = blockIdx.x * (blockDim.x / L) + tid / L;
+  const bool active = col < cols;
+  const int g = h / (a.H / a.G), Kd = a.G * dk, C = 2 * Kd + a.H * dv;
+  float* state = a.state + (int64_t)slot * a.state_stride + (int64_t)h * rows * cols;
+  f32x2 S[ROWS / 2], bonus[ROWS / 2];
+  load_state(state, cols, col, active, part, dk, S);
+  if (RULE == RULE_WKV) load_state(a.bonus + h * dk, 1, 0, true, part, dk, bonus);
+  float m_run = 0.f;
+  if (RULE == RULE_MLSTM && active) m_run = state[(int64_t)dk * cols + col];
+
+  const int wide = !DELTA && a.bf16;
+  const bool whole = a.pieces && part * ROWS + ROWS <= dk;       // 16 channels on 16-byte boundaries
+  // channels part * ROWS ... of a row that starts at element `at`, as register pairs (zeros past dk)
+  auto channels = [&](const void* base, int64_t at, int bf16, ulonglong2 (&to)[ROWS / 4]) {
+    at += part * ROWS;
+    if (whole && bf16) {
+      const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(base) + at);
+#pragma unroll
+      for (int r = 0; r < ROWS / 8; ++r) {
+        const uint4 v = src[r];
+        to[2 * r].x = pack2(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u));
+        to[2 * r].y = pack2(__uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+        to[2 * r + 1].x = pack2(__uint_as_float(v.z << 16), __uint_as_float(v.z & 0xffff0000u));
+        to[2 * r + 1].y = pack2(__uint_as_float(v.w << 16), __uint_as_float(v.w & 0xffff0000u));
+      }
+    } else if (whole) {
+      const ulonglong2* src = reinterpret_cast<const ulonglong2*>(reinterpret_cast<const float*>(base) + at);
+#pragma unroll
+      for (int r = 0; r < ROWS / 4; ++r) to[r] = src[r];
+    } else {
+      auto value = [&](int i) { return part * ROWS + i < dk ? engine_value(base, at + i, bf16) : 0.f; };
+#pragma unroll
+      for (int r = 0; r < ROWS / 4; ++r) {
+        to[r].x = pack2(value(4 * r), value(4 * r + 1));
+        to[r].y = pack2(value(4 * r + 2), value(4 * r + 3));
+      }
+    }
+  };
+  for (int tt = 0; tt < n; ++tt) {
+    const int64_t t = t0 + tt;
+    TokenRows rows_of;
+    float v = 0.f, beta = 0.f, keep = 0.f, floor = 0.f;
+    if constexpr (DELTA) {
+      channels(a.in_a, t * C + g * dk, 0, rows_of.a);
+      channels(a.in_a, t * C + Kd + g * dk, 0, rows_of.b);
+      if (active) v = reinterpret_cast<const float*>(a.in_a)[t * C + 2 * Kd + h * dv + col];
+      beta = a.beta[t * a.H + h];
+      if (ONE_DECAY) keep = a.decay[t * a.H + h];
+    } else {
+      const int64_t k_ld = COLUMNS ? a.in_ld : (int64_t)a.H * dk, v_ld = COLUMNS ? a.in_ld : (int64_t)a.H * dv;
+      channels(a.in_a, t * k_ld + h * dk, wide, rows_of.a);
+      channels(a.in_b, t * k_ld + h * dk, wide, rows_of.b);
+      if (RULE == RULE_MLSTM && col == dv) v = 1.f;
+      else if (active) v = engine_value(a.in_v, t * v_ld + h * dv + col, wide);
+    }
+    if (!ONE_DECAY) channels(a.decay, t * a.decay_ld + h * dk, 0, rows_of.d);
+    if constexpr (RULE == RULE_MLSTM) {
+      const float* z = a.decay + t * 2 * a.H + h;
+      const float li = log_input_gate(z[0], a.gate_bias[h], a.gate_cap);
+      const float decayed = log_forget_gate(z[a.H], a.gate_bias[a.H + h], a.gate_cap) + m_run;
+      m_run = fmaxf(decayed, li);
+      v *= expf(li - m_run);
+      keep = expf(decayed - m_run);
+      floor = expf(-m_run);
+    }
+    float o = advance<RULE, L>(S, bonus, rows_of, v, beta, keep);
+#pragma unroll
+    for (int off = L >> 1; off > 0; off >>= 1) o += __shfl_xor_sync(0xffffffffu, o, off);
+    if (COLUMNS) o *= a.out_scale;
+    if (active && part == 0) {
+      float* dst = a.out + (t * a.H + h) * out_cols + col;
+      dst[0] = o;
+      if (RULE == RULE_MLSTM && col == dv) dst[1] = floor;
+    }
+  }
+  if (active) {
+    store_state(state, cols, col, part, dk, S);
+    if (RULE == RULE_MLSTM && part == 0) state[(int64_t)dk * cols + col] = m_run;
+  }
+  if (blockIdx.x == 0 && blockIdx.y == 0 && a.carry_rows > 0) carry_inputs(a, slot, t0, n);
+}
+
+template <int RULE, int L>
+int launch_step(RuleArgs& a, int max_portions, cudaStream_t stream) {
+  const int cols = RULE == RULE_MLSTM ? a.dv + 1 : a.dv;
+  int threads = STEP_THREADS;
+  while (threads > 32 && (threads / 2) / L >= cols) threads /= 2;
+  const int cb = threads / L;
+  cudaError_t e = ls_launch(rule_step_kernel<RULE, L>, dim3((cols + cb - 1) / cb, a.H, max_portions), dim3(threads), 0, stream, a);
+  if (e != cudaSuccess) return (int)e;
+  return ls_launch_status();
+}
+
+template <int RULE, int L>
+int launch_walk(RuleArgs& a, int max_portions, cudaStream_t stream) {
   const int cols = RULE == RULE_MLSTM ? a.dv + 1 : a.dv;
   const int per_warp = 32 / L, needed = (cols + per_warp - 1) / per_warp;      // columns of a warp, warps of a head
-  // Walking warps a block: four, or as many as the head needs.  A step with longer portions has few blocks and many tokens
-  // each: as few warps a block as give every SM one block, so that a walk is issued without a rival.
-  int warps = MAX_WALK_WARPS;
-  while (warps > 1 && warps / 2 >= needed) warps /= 2;
-  if (!SHORT) {
-    warps = 1;
-    while (warps < MAX_WALK_WARPS && warps < needed && (long long)a.H * ((needed + warps - 1) / warps) > 148) warps *= 2;
-  }
+  // Walking warps a block: few blocks have many tokens each, so as few warps a block as give every SM one block (a walk is
+  // then issued without a rival)
+  int warps = 1;
+  while (warps < MAX_WALK_WARPS && warps < needed && (long long)a.H * ((needed + warps - 1) / warps) > 148) warps *= 2;
   // (a chunk's values of that many columns are what the staging threads copy ahead)
   while (warps > 1 && (32 * warps / L + 2) * CHUNK > SINGLES * STAGERS) warps /= 2;
   a.walkers = 32 * warps;
@@ -607,19 +737,19 @@ int launch_as(RuleArgs& a, int max_portions, cudaStream_t stream) {
   if (smem > MOST_SMEM) return LS_E_SMEM;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(rule_kernel<RULE, L, SHORT>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST_SMEM) != cudaSuccess)
+    if (cudaFuncSetAttribute(rule_kernel<RULE, L>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST_SMEM) != cudaSuccess)
       return LS_E_SMEM;
     configured = true;
   }
   const dim3 grid((cols + cb - 1) / cb, a.H, max_portions);
-  cudaError_t e = ls_launch(rule_kernel<RULE, L, SHORT>, grid, dim3(a.walkers + STAGERS + (RULE == RULE_MLSTM ? 32 : 0)), smem, stream, a);
+  cudaError_t e = ls_launch(rule_kernel<RULE, L>, grid, dim3(a.walkers + STAGERS + (RULE == RULE_MLSTM ? 32 : 0)), smem, stream, a);
   if (e != cudaSuccess) return (int)e;
   return ls_launch_status();
 }
 
 template <int RULE, int L>
 int launch(RuleArgs& a, int tokens, int max_portions, cudaStream_t stream) {
-  return tokens <= max_portions ? launch_as<RULE, L, true>(a, max_portions, stream) : launch_as<RULE, L, false>(a, max_portions, stream);
+  return tokens <= max_portions ? launch_step<RULE, L>(a, max_portions, stream) : launch_walk<RULE, L>(a, max_portions, stream);
 }
 
 template <int RULE>
