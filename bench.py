@@ -578,7 +578,7 @@ def kernel_times(runner, entries_of, steps=3):
              "experts_product_tc", "experts_gather", "experts_combine", "latent_finish", "heads_product",
              "sigmoid_power_decay", "clamped_glu", "row_bias", "weighted_sum", "gated_sum", "experts_mix", "rmsnorm_shift", "experts_route_plan",
              "layernorm", "norm_merge_add", "pair_embed", "rows_cast", "scale_cap", "unit_gates", "unit_scan", "rotate_rows",
-             "side_gate"]
+             "side_gate", "side_gate_few"]
     records, saved, graphs, turn = [], {}, runner.graphs, [0]
     runner.graphs = None
 

@@ -74,7 +74,7 @@ enum LsKernelId {
   LS_K_CLAMPED_GLU, LS_K_ROW_BIAS, LS_K_WEIGHTED_SUM, LS_K_GLA_RULE, LS_K_SIGMOID_POWER_DECAY, LS_K_LATENT_FINISH,
   LS_K_HEADS_PRODUCT, LS_K_GATED_SUM, LS_K_EXPERTS_MIX, LS_K_RMSNORM_SHIFT,
   LS_K_LAYERNORM, LS_K_NORM_MERGE_ADD, LS_K_PAIR_EMBED, LS_K_ROWS_CAST, LS_K_SCALE_CAP, LS_K_UNIT_GATES, LS_K_UNIT_SCAN,
-  LS_K_ROTATE_ROWS, LS_K_DELTA_HEAD_RULE, LS_K_MLSTM_RULE, LS_K_SIDE_GATE,
+  LS_K_ROTATE_ROWS, LS_K_DELTA_HEAD_RULE, LS_K_MLSTM_RULE, LS_K_SIDE_GATE, LS_K_SIDE_GATE_FEW,
   LS_K_COUNT
 };
 #define LS_KERNEL_NAMES                                                                                  \
@@ -86,7 +86,7 @@ enum LsKernelId {
   "experts_gather,experts_up_tc,experts_down_tc,tanh_rows,double_exp_decay,"                      \
   "clamped_glu,row_bias,weighted_sum,gla_rule,sigmoid_power_decay,latent_finish,heads_product,"  \
   "gated_sum,experts_mix,rmsnorm_shift,layernorm,norm_merge_add,pair_embed,rows_cast,scale_cap,unit_gates,"                 \
-  "unit_scan,rotate_rows,delta_head_rule,mlstm_rule,side_gate"
+  "unit_scan,rotate_rows,delta_head_rule,mlstm_rule,side_gate,side_gate_few"
 // one table per library: hidden, so that two libraries loaded into one process do not share it
 __attribute__((visibility("hidden"))) inline unsigned long long ls_kernel_launches[LS_K_COUNT];
 #define LS_COUNT(id) (++ls_kernel_launches[id])

@@ -89,7 +89,7 @@ __device__ __forceinline__ int tokens_before(const int* __restrict__ token_slot,
 }
 
 // ---------------------------------------------------------------------------------------
-// gated delta rule: everything between the projections and the recurrence, one block a token
+// gated delta rule: everything between the projections and the recurrence
 // ---------------------------------------------------------------------------------------
 constexpr int PREP_THREADS = 256;
 
@@ -112,57 +112,72 @@ struct DeltaPrepArgs {
   const float* gates;
 };
 
+constexpr int PREP_WARPS = PREP_THREADS / 32;
+constexpr int PREP_COLUMNS = 8;    // channels of a warp's segment that a lane has at most (heads up to 256)
+constexpr int PREP_SEGMENT = 128;  // channels of a segment that is no head
+
+// A warp has a segment of one token: a head of q or of k, 128 channels of v, 128 channels of the decay, or the token's
+// numbers per head.
 template <typename T>
-__global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(DeltaPrepArgs a) {
-  extern __shared__ float smem[];
+__global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(DeltaPrepArgs a, int v_segments) {
   ls_dependency_sync();
-  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int t = blockIdx.x, lane = threadIdx.x & 31;
+  int segment = blockIdx.y * PREP_WARPS + (threadIdx.x >> 5);
   const int Kd = a.G * a.dk, Vd = a.H * a.dv, C = 2 * Kd + Vd;
-  float* conv = smem;              // [C]
-  float* head_scale = conv + C;    // [2 G]
   const T* proj = reinterpret_cast<const T*>(a.proj);
   const T* row = proj + (int64_t)t * a.ld;
-  const int slot = a.token_slot[t];
-  const int before = tokens_before(a.token_slot, t, a.taps - 1);
-  const float* carried = a.state + (int64_t)slot * a.state_stride + (int64_t)a.H * a.dk * a.dv;
-
-  for (int c = tid; c < C; c += PREP_THREADS) {
-    float acc = 0.f;
-    for (int j = 0; j < a.taps; ++j) {
-      const int back = a.taps - 1 - j;
-      float x;
-      if (back <= before) x = ls_to_float<T>(proj[(int64_t)(t - back) * a.ld + c]);
-      else x = carried[(int64_t)(a.taps - 2 - (back - before - 1)) * C + c];
-      acc = fmaf(a.conv_w[c * a.taps + j], x, acc);
-    }
-    conv[c] = silu_f(acc);
-  }
-  __syncthreads();
-  // q and k heads to unit length; q also by dk^(-1/2)
-  for (int h = warp; h < 2 * a.G; h += PREP_THREADS / 32) {
+  if (segment < 2 * a.G + v_segments) {
+    const int slot = a.token_slot[t];
+    const int before = tokens_before(a.token_slot, t, a.taps - 1);
+    const float* carried = a.state + (int64_t)slot * a.state_stride + (int64_t)a.H * a.dk * a.dv;
+    const bool head = segment < 2 * a.G;
+    const int first = head ? segment * a.dk : 2 * Kd + (segment - 2 * a.G) * PREP_SEGMENT;
+    const int count = head ? a.dk : (C - first < PREP_SEGMENT ? C - first : PREP_SEGMENT);
+    float v[PREP_COLUMNS];
     float ss = 0.f;
-    for (int i = lane; i < a.dk; i += 32) {
-      const float v = conv[h * a.dk + i];
-      ss = fmaf(v, v, ss);
+#pragma unroll
+    for (int m = 0; m < PREP_COLUMNS; ++m) {
+      const int i = lane + 32 * m, c = first + i;
+      v[m] = 0.f;
+      if (i >= count) continue;
+      float acc = 0.f;
+#pragma unroll 4
+      for (int j = 0; j < a.taps; ++j) {
+        const int back = a.taps - 1 - j;
+        const float x = back <= before ? ls_to_float<T>(row[c - (int64_t)back * a.ld])
+                                       : carried[(int64_t)(a.taps - 2 - (back - before - 1)) * C + c];
+        acc = fmaf(a.conv_w[c * a.taps + j], x, acc);
+      }
+      v[m] = silu_f(acc);
+      ss = fmaf(v[m], v[m], ss);
     }
-    ss = ls_warp_sum(ss);
-    if (lane == 0) head_scale[h] = (1.0f / sqrtf(ss + a.unit_eps)) * (h < a.G ? 1.0f / sqrtf((float)a.dk) : 1.0f);
+    // q and k heads to unit length; q also by dk^(-1/2)
+    float scale = 1.0f;
+    if (head) scale = (1.0f / sqrtf(ls_warp_sum(ss) + a.unit_eps)) * (segment < a.G ? 1.0f / sqrtf((float)a.dk) : 1.0f);
+    float* out = a.qkv + (int64_t)t * C + first;
+#pragma unroll
+    for (int m = 0; m < PREP_COLUMNS; ++m)
+      if (lane + 32 * m < count) out[lane + 32 * m] = head ? v[m] * scale : v[m];
+    return;
   }
-  __syncthreads();
-  float* out = a.qkv + (int64_t)t * C;
-  for (int c = tid; c < C; c += PREP_THREADS) out[c] = c < 2 * Kd ? conv[c] * head_scale[c / a.dk] : conv[c];
-  if (a.gates != nullptr) {
+  segment -= 2 * a.G + v_segments;
+  if (segment == 0) {
     const float* z = a.gates + (int64_t)t * 2 * a.H;
-    for (int h = tid; h < a.H; h += PREP_THREADS) {
-      a.beta[(int64_t)t * a.H + h] = sigmoid_f(z[h]);
-      a.decay[(int64_t)t * a.H + h] = expf(-expf(a.a_log[h]) * softplus_f(z[a.H + h] + a.dt_bias[h]));
+    for (int h = lane; h < a.H; h += 32) {
+      a.beta[(int64_t)t * a.H + h] = sigmoid_f(a.gates != nullptr ? z[h] : ls_to_float<T>(row[C + h]));
+      if (a.gates != nullptr)
+        a.decay[(int64_t)t * a.H + h] = expf(-expf(a.a_log[h]) * softplus_f(z[a.H + h] + a.dt_bias[h]));
     }
     return;
   }
-  for (int h = tid; h < a.H; h += PREP_THREADS) a.beta[(int64_t)t * a.H + h] = sigmoid_f(ls_to_float<T>(row[C + h]));
-  float* decay = a.decay + (int64_t)t * a.H * a.dk;
-  for (int i = tid; i < a.H * a.dk; i += PREP_THREADS)
-    decay[i] = expf(-expf(a.a_log[i / a.dk]) * softplus_f(decay[i] + a.dt_bias[i]));
+  // a decay per channel
+  const int channels = a.gates != nullptr ? 0 : a.H * a.dk;
+  float* decay = a.decay + (int64_t)t * channels;
+#pragma unroll
+  for (int m = 0; m < PREP_SEGMENT / 32; ++m) {
+    const int i = (segment - 1) * PREP_SEGMENT + lane + 32 * m;
+    if (i < channels) decay[i] = expf(-expf(a.a_log[i / a.dk]) * softplus_f(decay[i] + a.dt_bias[i]));
+  }
 }
 
 // z <- exp(-exp(z + bias[column])), element by element: a decay from its low-rank map's output
@@ -269,17 +284,16 @@ LS_API int ls_delta_prep(const void* proj, int64_t ld, int dtype, const float* c
   a.proj = proj; a.ld = ld; a.conv_w = conv_w; a.dt_bias = dt_bias; a.a_log = a_log; a.state = state;
   a.state_stride = state_stride; a.token_slot = token_slot; a.qkv = qkv; a.decay = decay; a.beta = beta; a.T = tokens;
   a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.taps = taps; a.unit_eps = unit_eps;
-  const size_t smem = sizeof(float) * (size_t)(2 * G * dk + H * dv + 2 * G);
-  if (smem > 200 * 1024) return LS_E_SMEM;
+  if (dk > 32 * PREP_COLUMNS) return LS_E_SIZE;
+  const int v_segments = (H * dv + PREP_SEGMENT - 1) / PREP_SEGMENT;
+  const int segments = 2 * G + v_segments + 1 + (gates != nullptr ? 0 : (H * dk + PREP_SEGMENT - 1) / PREP_SEGMENT);
+  const dim3 grid(tokens, (segments + PREP_WARPS - 1) / PREP_WARPS);
+  if (grid.y > 65535) return LS_E_SIZE;
   LS_COUNT(LS_K_DELTA_PREP);
   cudaError_t e;
-  if (dtype == LS_F32) {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    e = ls_launch(delta_prep_kernel<float>, dim3(tokens), dim3(PREP_THREADS), smem, stream, a);
-  } else if (dtype == LS_BF16) {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prep_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    e = ls_launch(delta_prep_kernel<__nv_bfloat16>, dim3(tokens), dim3(PREP_THREADS), smem, stream, a);
-  } else return LS_E_DTYPE;
+  if (dtype == LS_F32) e = ls_launch(delta_prep_kernel<float>, grid, dim3(PREP_THREADS), 0, stream, a, v_segments);
+  else if (dtype == LS_BF16) e = ls_launch(delta_prep_kernel<__nv_bfloat16>, grid, dim3(PREP_THREADS), 0, stream, a, v_segments);
+  else return LS_E_DTYPE;
   if (e != cudaSuccess) return (int)e;
   return ls_launch_status();
 }

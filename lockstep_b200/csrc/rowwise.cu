@@ -8,7 +8,8 @@
 //     token and the one before it, whose last row serves a sequence's first token;
 //   - float32 rows written into some columns of a wider row of the engine's type; logits times a
 //     factor, then capped with tanh;
-//   - the gate of a token's own embedding in a layer: gelu(z) times some columns of the token's row of a table.
+//   - the gate of a token's own embedding in a layer: gelu(z) times some columns of the token's row of a table; for few
+//     tokens with the product that makes z in the same kernel.
 // All reductions run in float32 in an order fixed by the row's own width (a thread's elements
 // ascending, the lanes by an xor tree, the warps ascending), so a row's result does not depend on the batch.
 #include "common.cuh"
@@ -208,6 +209,79 @@ __global__ void side_gate_kernel(const float* __restrict__ z, const int* __restr
   }
 }
 
+// The same with z[t, c] = h[t, :] . w[c, :] made here, for few tokens: a block has SIDE_ROWS rows of w and up to SIDE_TOKENS
+// tokens, a thread every 128th piece of eight elements of all of them (a sum is a chain per thread over its pieces; the
+// threads' sums are added sixteen at a time, then by an xor tree over eight lanes).
+constexpr int SIDE_TOKENS = 8, SIDE_ROWS = 2, SIDE_THREADS = 128;
+
+__global__ void __launch_bounds__(SIDE_THREADS)
+side_gate_few_kernel(const float* __restrict__ h, const __nv_bfloat16* __restrict__ w, const int* __restrict__ ids,
+                     const __nv_bfloat16* __restrict__ table, int64_t table_ld, int at, int vocab,
+                     __nv_bfloat16* __restrict__ out, int tokens, int width, int dim, int* err) {
+  __shared__ float sums[SIDE_ROWS * SIDE_TOKENS][SIDE_THREADS + 1];
+  ls_dependency_trigger();
+  const int tid = threadIdx.x, c0 = blockIdx.x * SIDE_ROWS, t0 = blockIdx.y * SIDE_TOKENS;
+  const int left = tokens - t0 < SIDE_TOKENS ? tokens - t0 : SIDE_TOKENS;
+  float acc[SIDE_ROWS][SIDE_TOKENS];
+#pragma unroll
+  for (int r = 0; r < SIDE_ROWS; ++r)
+#pragma unroll
+    for (int m = 0; m < SIDE_TOKENS; ++m) acc[r][m] = 0.f;
+  ls_dependency_wait();
+  for (int k = tid * 8; k < width; k += 8 * SIDE_THREADS) {
+    // (rows past the last one are read again: the loads of a piece go out together)
+    uint4 raw[SIDE_ROWS];
+    float4 lo[SIDE_TOKENS], hi[SIDE_TOKENS];
+#pragma unroll
+    for (int r = 0; r < SIDE_ROWS; ++r)
+      raw[r] = *reinterpret_cast<const uint4*>(w + (int64_t)(c0 + r < dim ? c0 + r : dim - 1) * width + k);
+#pragma unroll
+    for (int m = 0; m < SIDE_TOKENS; ++m) {
+      const float4* src = reinterpret_cast<const float4*>(h + (int64_t)(t0 + (m < left ? m : left - 1)) * width + k);
+      lo[m] = src[0];
+      hi[m] = src[1];
+    }
+#pragma unroll
+    for (int r = 0; r < SIDE_ROWS; ++r) {
+      const float wf[8] = {__uint_as_float(raw[r].x << 16), __uint_as_float(raw[r].x & 0xffff0000u), __uint_as_float(raw[r].y << 16),
+                           __uint_as_float(raw[r].y & 0xffff0000u), __uint_as_float(raw[r].z << 16),
+                           __uint_as_float(raw[r].z & 0xffff0000u), __uint_as_float(raw[r].w << 16),
+                           __uint_as_float(raw[r].w & 0xffff0000u)};
+#pragma unroll
+      for (int m = 0; m < SIDE_TOKENS; ++m) {
+        float& s = acc[r][m];
+        s = fmaf(lo[m].x, wf[0], s); s = fmaf(lo[m].y, wf[1], s); s = fmaf(lo[m].z, wf[2], s); s = fmaf(lo[m].w, wf[3], s);
+        s = fmaf(hi[m].x, wf[4], s); s = fmaf(hi[m].y, wf[5], s); s = fmaf(hi[m].z, wf[6], s); s = fmaf(hi[m].w, wf[7], s);
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < SIDE_ROWS; ++r)
+#pragma unroll
+    for (int m = 0; m < SIDE_TOKENS; ++m) sums[r * SIDE_TOKENS + m][tid] = acc[r][m];
+  __syncthreads();
+  // eight lanes an output
+  const int o = tid >> 3, sub = tid & 7;
+  static_assert(SIDE_THREADS == 8 * SIDE_ROWS * SIDE_TOKENS, "eight lanes an output");
+  float z = 0.f;
+#pragma unroll
+  for (int i = 0; i < SIDE_THREADS / 8; ++i) z += sums[o][sub + 8 * i];
+  z += __shfl_xor_sync(0xffffffffu, z, 4);
+  z += __shfl_xor_sync(0xffffffffu, z, 2);
+  z += __shfl_xor_sync(0xffffffffu, z, 1);
+  const int c = c0 + o / SIDE_TOKENS, m = o % SIDE_TOKENS;
+  if (sub == 0 && c < dim && m < left) {
+    const int t = t0 + m, id = ids[t];
+    float v = 0.f;
+    if (id < 0 || id >= vocab) {
+      if (c == 0) ls_record_fault(err, LS_DEV_TOKEN_RANGE, t);
+    } else {
+      v = ls_gelu_tanh(z) * __bfloat162float(table[id * table_ld + at + c]);
+    }
+    out[(int64_t)t * dim + c] = __float2bfloat16_rn(v);
+  }
+}
+
 inline int blocks_for(int64_t n) { return (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16); }
 
 }  // namespace
@@ -293,6 +367,19 @@ LS_API int ls_side_gate(const float* z, const int* ids, const void* table, long 
     ls_launch(side_gate_kernel<__nv_bfloat16>, blocks_for(tokens * dim), 256, 0, stream, z, ids, (const __nv_bfloat16*)table,
               (int64_t)table_ld, at, vocab, (__nv_bfloat16*)out, (int64_t)tokens, dim, err);
   else return LS_E_DTYPE;
+  return ls_launch_status();
+}
+
+// bfloat16 weights, table and output; the width a multiple of 8, rows on 16-byte boundaries (else LS_E_ALIGN, nothing launched).
+LS_API int ls_side_gate_few(const float* h, const void* w, const int* ids, const void* table, long long table_ld, int at,
+                            int vocab, void* out, int tokens, int width, int dim, int* err, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (dim <= 0 || width <= 0 || at < 0 || at + dim > table_ld || vocab <= 0) return LS_E_SIZE;
+  if (width % 8 || ((uintptr_t)h & 15) || ((uintptr_t)w & 15)) return LS_E_ALIGN;
+  LS_COUNT(LS_K_SIDE_GATE_FEW);
+  const dim3 grid((dim + SIDE_ROWS - 1) / SIDE_ROWS, (tokens + SIDE_TOKENS - 1) / SIDE_TOKENS);
+  ls_launch(side_gate_few_kernel, grid, dim3(SIDE_THREADS), 0, stream, h, (const __nv_bfloat16*)w, ids,
+            (const __nv_bfloat16*)table, (int64_t)table_ld, at, vocab, (__nv_bfloat16*)out, tokens, width, dim, err);
   return ls_launch_status();
 }
 

@@ -58,7 +58,7 @@ struct RuleArgs {
   const float* beta;       // delta
   const float* bonus;      // wkv
   float* out;              // [T, H dv] float32 (mlstm: [T, H (dv + 2)])
-  // what else the state carries, updated by one block per portion after the walk
+  // what else the state carries, brought up to date after the walk
   const void* carry_src;   // delta: the raw projection [T, ld] (its first C columns); wkv: the mixer's input [T, width]
   int64_t carry_ld;
   int carry_width;         // delta: C; wkv: width
@@ -216,11 +216,13 @@ __device__ __forceinline__ void store_state(float* state, int cols, int col, int
   }
 }
 
-// The rest of the state: the last inputs of a portion (its first token t0, n tokens), behind those that were carried.
+// The rest of the state: the last inputs of a portion (its first token t0, n tokens), behind those that were carried.  All
+// blocks of the portion share the channels.
 __device__ __forceinline__ void carry_inputs(const RuleArgs& a, int slot, int t0, int n) {
   float* carried = a.state + (int64_t)slot * a.state_stride + (int64_t)a.H * a.dk * a.dv;
   const int rows = a.carry_rows, W = a.carry_width;
-  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+  const int block = blockIdx.y * gridDim.x + blockIdx.x, blocks = gridDim.x * gridDim.y;
+  for (int c = block * blockDim.x + threadIdx.x; c < W; c += blocks * blockDim.x) {
     float keep[MAX_TAPS];
     for (int s = 0; s < rows; ++s) {
       const int from = n - rows + s;
@@ -599,7 +601,7 @@ rule_kernel(RuleArgs a) {
     if (RULE == RULE_MLSTM) meet();
   }
 
-  if (blockIdx.x == 0 && blockIdx.y == 0 && a.carry_rows > 0) carry_inputs(a, slot, t0, n);
+  if (a.carry_rows > 0) carry_inputs(a, slot, t0, n);
 }
 
 // Steps of single tokens: every thread fetches what it needs of a token itself, beside its part of the state (nothing is
@@ -697,7 +699,7 @@ __global__ void __launch_bounds__(STEP_THREADS, 4) rule_step_kernel(RuleArgs a) 
     store_state(state, cols, col, part, dk, S);
     if (RULE == RULE_MLSTM && part == 0) state[(int64_t)dk * cols + col] = m_run;
   }
-  if (blockIdx.x == 0 && blockIdx.y == 0 && a.carry_rows > 0) carry_inputs(a, slot, t0, n);
+  if (a.carry_rows > 0) carry_inputs(a, slot, t0, n);
 }
 
 template <int RULE, int L>

@@ -62,6 +62,8 @@ _SIGNATURES = {
         "ls_scale_cap": [c_void_p, ctypes.c_longlong, c_float, c_float, c_void_p],
         "ls_side_gate": [c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int, c_void_p, c_int, ctypes.c_longlong,
                          c_int, c_void_p, c_void_p],
+        "ls_side_gate_few": [c_void_p, c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_int, c_int, c_void_p, c_int, c_int,
+                             c_int, c_void_p, c_void_p],
         "ls_row_bias": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "ls_weighted_sum": [c_void_p, c_void_p, ctypes.c_longlong, c_int, ctypes.POINTER(c_float), c_void_p, c_int,
                             c_void_p],
@@ -511,6 +513,23 @@ def side_gate(z, ids, table, at: int, out, err) -> None:
         table.shape[0], _dev(out, "out"), _code(out), tokens, dim, _dev(err, "err", torch.int32), _stream()), "side_gate")
 
 
+def side_gate_few(h, w, ids, table, at: int, out, err) -> bool:
+    """``side_gate`` with z = h @ w.T made in the same kernel, for few tokens: ``h`` float32 [tokens, width], the others
+    bfloat16.  Returns False, having launched nothing, for rows it cannot read in pieces."""
+    tokens, dim = out.shape
+    if tuple(w.shape) != (dim, h.shape[1]) or h.shape[0] != tokens or ids.numel() != tokens or at + dim > table.shape[1]:
+        raise KernelError("side_gate_few: shapes do not agree")
+    bf16 = torch.bfloat16
+    status = library().ls_side_gate_few(
+        _dev(h, "h", torch.float32), _dev(w, "w", bf16), _dev(ids, "ids", torch.int32), _dev(table, "table", bf16),
+        table.shape[1], int(at), table.shape[0], _dev(out, "out", bf16), tokens, h.shape[1], dim, _dev(err, "err", torch.int32),
+        _stream())
+    if status == -3:
+        return False
+    _check(status, "side_gate_few")
+    return True
+
+
 def _rows(t: torch.Tensor, name: str) -> tuple[int, int]:
     """(pointer, row pitch in elements) of a 2-D operand whose rows are contiguous: a whole
     tensor, or a view of some columns of one."""
@@ -904,7 +923,7 @@ def find_portions(token_slot, out, cap: int, err) -> None:
 
 def delta_prep(proj, conv_w, dt_bias, a_log, state, token_slot, qkv, decay, beta, heads: int, groups: int, dk: int,
                dv: int, taps: int, unit_eps: float, gates=None) -> None:
-    """What lies between the projections and the gated delta rule, a token a block: causal
+    """What lies between the projections and the gated delta rule: causal
     convolution (carried inputs from ``state``) and silu of q, k, v, unit q and k (q scaled),
     beta = sigmoid of its column, and the decay per key channel, made in place from the output
     of its low-rank map: ``decay`` <- exp(-exp(a_log[head]) softplus(decay + dt_bias)).  float32 out.

@@ -52,14 +52,18 @@ class TokenInput(Part):
 
     def forward(self, h: torch.Tensor, ctx) -> None:
         rt, tokens = self.rt, h.shape[0]
-        x = h
-        if rt.dtype != torch.float32:
-            x = rt.rows(tokens, self.w)
-            K.rows_cast(h, x)
-        z = rt.rows(tokens, self.dim, dtype=torch.float32)
-        K.gemm_nt(x, self.w_gate, z, err=rt.err)
+        table = rt.shared[self.table].table
         g = rt.rows(tokens, self.dim)
-        K.side_gate(z, ctx.token_ids, rt.shared[self.table].table, self.at, g, rt.err)
+        # few tokens: the gate's product, its activation and the token's row in one kernel
+        if not (rt.dtype == torch.bfloat16 and tokens <= K.FEW_TOKENS
+                and K.side_gate_few(h, self.w_gate, ctx.token_ids, table, self.at, g, rt.err)):
+            x = h
+            if rt.dtype != torch.float32:
+                x = rt.rows(tokens, self.w)
+                K.rows_cast(h, x)
+            z = rt.rows(tokens, self.dim, dtype=torch.float32)
+            K.gemm_nt(x, self.w_gate, z, err=rt.err)
+            K.side_gate(z, ctx.token_ids, table, self.at, g, rt.err)
         y = rt.rows(tokens, self.w, dtype=torch.float32)
         K.gemm_nt(g, self.w_proj, y, err=rt.err)
         K.norm_merge_add(h, y.view(1, tokens, self.w), self.gain, 1.0, None, self.eps, 0.0)

@@ -365,10 +365,13 @@ def test_token_input(dtype, tokens, width, dim):
     ctx.token_ids = torch.tensor(ids, dtype=torch.int32, device=DEV)
     h = torch.randn(tokens, width, device=DEV) * 2
     x = d64(h)
+    before = K.kernel_counts()
     part.forward(h, ctx)
     K.raise_on_fault(err)
     want = x + plain.token_side(x, ids, {k: d64(v) for k, v in w.items()}, 1, dim, 1e-5)
     assert float((d64(h) - want).abs().max()) <= _tol(dtype) * (1 + float(want.abs().max()))
+    few = K.kernel_counts()["side_gate_few"] - before["side_gate_few"]
+    assert few == (1 if dtype == BF16 and tokens <= K.FEW_TOKENS and width % 8 == 0 else 0)
 
 
 # ---------------------------------------------------------------------------
