@@ -43,8 +43,9 @@ __device__ __forceinline__ void mma_bf16(float* d, const uint32_t* a, uint32_t b
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// HALVES = d / 64.  Shared memory of a warp: K [HALVES][32 keys][128 B], then V the same.
-template <int HALVES>
+// HALVES = d / 64.  Shared memory of a warp: K [HALVES][32 keys][128 B], then V the same.  EXTRAS: the instance that
+// knows a bias, a cap and kept first keys; the other one keeps their branches out of the loop over the scores.
+template <int HALVES, bool EXTRAS>
 __global__ void __launch_bounds__(WARPS * 32, 3)
 attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_bfloat16* __restrict__ q,
                             float* __restrict__ part_acc, float* __restrict__ part_ml,
@@ -52,6 +53,7 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
                             int table_stride, int nq, int nkv, int page_size, int num_pages, int window,
                             int keep_first, float scale, float softcap, const float* __restrict__ slopes,
                             const float* __restrict__ log_rates, int* err) {
+  const int kept = EXTRAS ? keep_first : 0;
   // The work list, the block table and every key older than this step's token are there
   // before the step's first kernel starts, so the first chunks are fetched while the kernel
   // before this one (which writes the token's own key and value, and q) still runs.
@@ -95,7 +97,7 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
   const int r0 = lane >> 2, cq = (lane & 3) * 2;   // this thread holds rows r0 and r0 + 8
   // a bias that grows with the logarithm of the distance, per query head (rows past the group: none)
   float bias_a[2] = {0.f, 0.f}, bias_b[2] = {0.f, 0.f};
-  if (log_rates != nullptr) {
+  if (EXTRAS && log_rates != nullptr) {
 #pragma unroll
     for (int r = 0; r < 2; ++r)
       if (r0 + 8 * r < nq / nkv) {
@@ -120,11 +122,12 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
     const int i = lane >> 2, b = lane & 3;
     if (i < n_iter && b < boxes) {
       const int c0 = s_lo + (i * WARPS + warp) * CHUNK;
-      if (c0 < s_hi && (c0 + CHUNK > row_lo || c0 < keep_first)) {
+      if (c0 < s_hi && (c0 + CHUNK > row_lo || (EXTRAS && c0 < kept))) {
         int key = c0 + b * rows_per_box;
         if (key >= s_hi) key = s_hi - 1;          // beyond the split's end: any page that exists
-        if (key >= keep_first && key < row_lo && key / page_size != row_lo / page_size)
-          key = keep_first > 0 ? 0 : row_lo;      // behind the window: pages may have been given back
+        // behind the window: pages may have been given back
+        if (!EXTRAS) { if (key < row_lo) key = row_lo; }
+        else if (key >= kept && key < row_lo && key / page_size != row_lo / page_size) key = kept > 0 ? 0 : row_lo;
         my_page = table_row[key / page_size];
         if (my_page < 0 || my_page >= num_pages) {
           ls_record_fault(err, LS_DEV_PAGE_RANGE, key);
@@ -159,7 +162,7 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
   auto chunk_start = [&](int i) { return s_lo + (i * WARPS + warp) * CHUNK; };
   auto chunk_live = [&](int i) {
     const int c0 = chunk_start(i);
-    return i < n_iter && c0 < s_hi && (c0 + CHUNK > row_lo || c0 < keep_first);
+    return i < n_iter && c0 < s_hi && (c0 + CHUNK > row_lo || (EXTRAS && c0 < kept));
   };
 
   int it = 0;
@@ -233,9 +236,10 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = c0 + nt * 8 + cq + (e & 1);
-        const bool keep = key < s_hi && ls_sees(key, row_lo, keep_first);
+        const bool keep = key < s_hi && (EXTRAS ? ls_sees(key, row_lo, kept) : key >= row_lo);
         // (log_rates: slopes[head] x ln(1 + log_rates[head] x distance) is taken off the score)
         s[nt][e] = !keep ? -CUDART_INF_F
+                   : !EXTRAS ? s[nt][e] * scale
                    : log_rates != nullptr ? s[nt][e] * scale - bias_a[e >> 1] * log1pf(bias_b[e >> 1] * (float)(pos - key))
                                           : ls_capped(s[nt][e] * scale, softcap);
         tile_max[e >> 1] = fmaxf(tile_max[e >> 1], s[nt][e]);
@@ -284,11 +288,11 @@ attention_decode_mma_kernel(const __grid_constant__ CUtensorMap map, const __nv_
     // Values of masked keys (past the row's last key, behind its window) are whatever
     // the page holds; their weight is 0, but 0 * inf is not: clear those rows.
     {
-      const int valid_hi = s_hi - c0, valid_lo = row_lo - c0, valid_kept = keep_first - c0;
+      const int valid_hi = s_hi - c0, valid_lo = row_lo - c0, valid_kept = kept - c0;
       if (valid_hi < CHUNK || valid_lo > 0) {
         for (int idx = lane; idx < HALVES * CHUNK * 8; idx += 32) {
           const int half = idx / (CHUNK * 8), key = (idx / 8) % CHUNK, ch = idx & 7;
-          if (key >= valid_hi || (key < valid_lo && key >= valid_kept))
+          if (key >= valid_hi || (key < valid_lo && (!EXTRAS || key >= valid_kept)))
             *reinterpret_cast<uint4*>(aligned + (v_smem - base) + half * HALF_BYTES + key * 128 + ch * 16) =
                 make_uint4(0u, 0u, 0u, 0u);
         }
@@ -381,7 +385,7 @@ EncodeTiled encode_fn() {
   return fn;
 }
 
-template <int HALVES>
+template <int HALVES, bool EXTRAS>
 int launch(const CUtensorMap& map, const void* q, float* part_acc, float* part_ml, const int* work,
            int n_work, const int* block_table, int table_stride, int nq, int nkv, int page_size,
            int num_pages, int window, int keep_first, float scale, float softcap, const float* slopes,
@@ -389,13 +393,13 @@ int launch(const CUtensorMap& map, const void* q, float* part_acc, float* part_m
   const size_t smem = (size_t)WARPS * 2 * HALVES * CHUNK * 128 + 128 + 16 * HALVES * 128 + 1024;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_decode_mma_kernel<HALVES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attention_decode_mma_kernel<HALVES, EXTRAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              (int)smem) != cudaSuccess)
       return LS_E_SMEM;
     configured = true;
   }
   dim3 grid(n_work, nkv);
-  LS_COUNT(LS_K_ATTENTION_DECODE_MMA), ls_launch(attention_decode_mma_kernel<HALVES>, grid, WARPS * 32, smem, stream, 
+  LS_COUNT(LS_K_ATTENTION_DECODE_MMA), ls_launch(attention_decode_mma_kernel<HALVES, EXTRAS>, grid, WARPS * 32, smem, stream, 
       map, (const __nv_bfloat16*)q, part_acc, part_ml, work, block_table, table_stride, nq, nkv, page_size,
       num_pages, window, keep_first, scale, softcap, slopes, log_rates, err);
   return ls_launch_status();
@@ -430,11 +434,10 @@ LS_API int ls_attention_decode_mma(const void* q, const void* pages, float* part
           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
     return LS_E_SIZE;
-  if (d == 64)
-    return launch<1>(map, q, part_acc, part_ml, work, n_work, block_table, table_stride, nq, nkv, page_size,
-                     num_pages, window, keep_first, scale, softcap, slopes, log_rates, err, stream);
-  return launch<2>(map, q, part_acc, part_ml, work, n_work, block_table, table_stride, nq, nkv, page_size,
-                   num_pages, window, keep_first, scale, softcap, slopes, log_rates, err, stream);
+  auto go = keep_first > 0 || softcap > 0.f || log_rates != nullptr ? (d == 64 ? launch<1, true> : launch<2, true>)
+                                                                    : (d == 64 ? launch<1, false> : launch<2, false>);
+  return go(map, q, part_acc, part_ml, work, n_work, block_table, table_stride, nq, nkv, page_size, num_pages, window,
+            keep_first, scale, softcap, slopes, log_rates, err, stream);
 }
 
 LS_API const char* ls_constants_attention_decode_mma() {
