@@ -114,7 +114,7 @@ class PagedGroup:
         if not self.window:
             return 0
         q = kv_len_after if first_query_pos is None else first_query_pos
-        lo = q - self.window + 1
+        lo = q - self.window + 1 if self.window > 0 else q - q % -self.window      # (< 0: chunks of -window positions)
         return max(0, lo) // self.page_size
 
     def readable(self, logical: int, pos: int) -> bool:
@@ -330,7 +330,7 @@ class CacheManager:
         for g in self.paged:
             need = -(-total_tokens // self.page_size)
             if g.window and total_tokens > max_portion:
-                need = min(need, -(-(g.window - 1 + max_portion) // self.page_size) + 1 + g.keep_boundary_window
+                need = min(need, -(-(abs(g.window) - 1 + max_portion) // self.page_size) + 1 + g.keep_boundary_window
                            + g.kept_pages)
             worst = max(worst, need)
         return worst

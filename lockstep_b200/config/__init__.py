@@ -15,9 +15,11 @@ from . import pikurax as _pikurax  # registers Pikurax
 from .pikurax import PikuraxConfig
 from . import kusolorn as _kusolorn  # registers Kusolorn
 from .kusolorn import KusolornConfig
+from . import tesozen as _tesozen  # registers Tesozen
+from .tesozen import TesozenConfig
 
 __all__ = [
-    "ConfigError", "KemiraxConfig", "KusolornConfig", "LayerRun", "LayerSpec", "MalazenConfig", "ModelSpec", "PartSpec", "PikuraxConfig", "Qwen3Config", "SevipelConfig",
+    "ConfigError", "KemiraxConfig", "KusolornConfig", "LayerRun", "LayerSpec", "MalazenConfig", "ModelSpec", "PartSpec", "PikuraxConfig", "Qwen3Config", "SevipelConfig", "TesozenConfig",
     "architecture_name", "config_from_dict", "known_architectures", "load_config",
     "own_tensors", "register_architecture", "tensor_name", "unregister_architecture",
 ]

@@ -75,6 +75,7 @@ enum LsKernelId {
   LS_K_HEADS_PRODUCT, LS_K_GATED_SUM, LS_K_EXPERTS_MIX, LS_K_RMSNORM_SHIFT,
   LS_K_LAYERNORM, LS_K_NORM_MERGE_ADD, LS_K_PAIR_EMBED, LS_K_ROWS_CAST, LS_K_SCALE_CAP, LS_K_UNIT_GATES, LS_K_UNIT_SCAN,
   LS_K_ROTATE_ROWS, LS_K_DELTA_HEAD_RULE, LS_K_MLSTM_RULE, LS_K_SIDE_GATE, LS_K_SIDE_GATE_FEW,
+  LS_K_MAP_DIFFERENCE, LS_K_MAP_DIFFERENCE_FOLD, LS_K_NORM_MERGE_NORM,
   LS_K_COUNT
 };
 #define LS_KERNEL_NAMES                                                                                  \
@@ -86,7 +87,8 @@ enum LsKernelId {
   "experts_gather,experts_up_tc,experts_down_tc,tanh_rows,double_exp_decay,"                      \
   "clamped_glu,row_bias,weighted_sum,gla_rule,sigmoid_power_decay,latent_finish,heads_product,"  \
   "gated_sum,experts_mix,rmsnorm_shift,layernorm,norm_merge_add,pair_embed,rows_cast,scale_cap,unit_gates,"                 \
-  "unit_scan,rotate_rows,delta_head_rule,mlstm_rule,side_gate,side_gate_few"
+  "unit_scan,rotate_rows,delta_head_rule,mlstm_rule,side_gate,side_gate_few,"   \
+  "map_difference,map_difference_fold,norm_merge_norm"
 // one table per library: hidden, so that two libraries loaded into one process do not share it
 __attribute__((visibility("hidden"))) inline unsigned long long ls_kernel_launches[LS_K_COUNT];
 #define LS_COUNT(id) (++ls_kernel_launches[id])
@@ -157,6 +159,12 @@ __device__ __forceinline__ float ls_capped(float score, float cap) {
 // the tanh form of gelu: 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
 __device__ __forceinline__ float ls_gelu_tanh(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+// the square of relu
+__device__ __forceinline__ float ls_relu_squared(float z) {
+  const float r = fmaxf(z, 0.f);
+  return r * r;
 }
 
 // Programmatic dependent launch: a kernel may be scheduled while its predecessor

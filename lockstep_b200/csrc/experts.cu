@@ -5,7 +5,8 @@
 // Router logits arrive as float32 [tokens, experts].  The score is the sigmoid of the logit, or
 // the softmax over all experts; the `top` largest scores (plus an optional correction per expert
 // that only the choice sees) are chosen (ties to the lower index) and kept in order of rank; the
-// weight is the score itself.  The last experts may be identities, which have no weights and no
+// weight is the score itself, or its share of the chosen scores' sum times a factor.  The choice may be
+// limited to the experts of the best few of equal groups of neighbours.  The last experts may be identities, which have no weights and no
 // rows in the sorted order: the sum takes the token's own row for them.  A pair's
 // row in the sorted order is handed out by a counter per expert, so which row a pair gets
 // may differ from run to run, but no value depends on it: every element of a product is one
@@ -14,6 +15,11 @@
 #include "common.cuh"
 
 namespace {
+
+struct RoutePick {
+  int groups, keep;
+  float factor;
+};
 
 constexpr int MAX_PER_LANE = 16;      // experts a lane looks after: up to 512 experts
 constexpr int ROUTE_WARPS = 8;
@@ -24,10 +30,13 @@ constexpr int TILE_M = 64, TILE_N = 64, TILE_K = 16;
 // softmax 0: weight = sigmoid(logit); 1: weight = softmax over the `experts` logits (the largest taken off, the
 // exponentials summed lane by lane over ascending experts, then by an xor tree: an order the token alone fixes).
 // correction (or null) [experts]: added to the weight for the choice only.
+// pick: groups > 0: only experts of the `keep` best of that many equal groups of neighbours can be chosen, a group's
+// score the sum of its two largest choice scores (ties to the lower group); factor > 0: the weights are divided by
+// (their sum over the chosen, in order of rank, + 1e-20) and multiplied by it.
 // (one warp: token t)
 __device__ __forceinline__ void route_token(const float* __restrict__ logits, int64_t ld, int t, int experts, int top,
-                                            int softmax, const float* __restrict__ correction, int* __restrict__ ids,
-                                            float* __restrict__ weights) {
+                                            int softmax, const float* __restrict__ correction, const RoutePick rule,
+                                            int* __restrict__ ids, float* __restrict__ weights) {
   const int lane = threadIdx.x & 31;
   float z[MAX_PER_LANE];     // the expert's score
   float pick[MAX_PER_LANE];  // what the choice compares
@@ -60,6 +69,65 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
   for (int i = 0; i < MAX_PER_LANE; ++i) {
     const int e = lane + 32 * i;
     pick[i] = e < experts ? (correction != nullptr ? z[i] + correction[e] : z[i]) : -INFINITY;
+  }
+  if (rule.groups > 0) {
+    // lane g % 32 keeps the score of group g in place g / 32; the choice then takes the best groups one by one
+    const int size = experts / rule.groups;
+    float group_score[MAX_PER_LANE];
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) group_score[i] = -INFINITY;
+    for (int g = 0; g < rule.groups; ++g) {
+      const int from = g * size, to = from + size;
+      float a = -INFINITY, b = -INFINITY;              // the largest and the second of this lane's experts of the group
+#pragma unroll
+      for (int i = 0; i < MAX_PER_LANE; ++i) {
+        const int e = lane + 32 * i;
+        if (e >= from && e < to) {
+          b = fmaxf(b, fminf(a, pick[i]));
+          a = fmaxf(a, pick[i]);
+        }
+      }
+      for (int off = 16; off > 0; off >>= 1) {
+        const float oa = __shfl_xor_sync(0xffffffffu, a, off);
+        const float ob = __shfl_xor_sync(0xffffffffu, b, off);
+        b = fmaxf(fminf(a, oa), fmaxf(b, ob));
+        a = fmaxf(a, oa);
+      }
+      const float score = size > 1 ? a + b : a;
+#pragma unroll
+      for (int i = 0; i < MAX_PER_LANE; ++i)
+        if (lane + 32 * i == g) group_score[i] = score;
+    }
+    unsigned open = 0;                                 // this lane's experts whose group is kept
+    for (int r = 0; r < rule.keep; ++r) {
+      float best = -INFINITY;
+      int at = 0x7fffffff;
+#pragma unroll
+      for (int i = 0; i < MAX_PER_LANE; ++i) {
+        const int g = lane + 32 * i;
+        if (g < rule.groups && (group_score[i] > best || (group_score[i] == best && g < at))) {
+          best = group_score[i];
+          at = g;
+        }
+      }
+      for (int off = 16; off > 0; off >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, off);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, off);
+        if (ob > best || (ob == best && oa < at)) {
+          best = ob;
+          at = oa;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < MAX_PER_LANE; ++i) {
+        const int e = lane + 32 * i;
+        if (e == at) group_score[i] = -INFINITY;       // (as a group: taken)
+        if (e >= at * size && e < (at + 1) * size) open |= 1u << i;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i)
+      if (!((open >> i) & 1u)) pick[i] = -INFINITY;
   }
   unsigned taken = 0;
   for (int r = 0; r < top; ++r) {
@@ -101,16 +169,22 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
     }
     for (int r = 0; r < top; ++r) w[r] = w[r] / sum;
   }
+  if (rule.factor > 0.f && lane == 0) {
+    float* w = weights + (int64_t)t * top;
+    float sum = 0.f;
+    for (int r = 0; r < top; ++r) sum += w[r];
+    for (int r = 0; r < top; ++r) w[r] = w[r] / (sum + 1e-20f) * rule.factor;
+  }
 }
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_kernel(const float* __restrict__ logits, int64_t ld, int tokens,
                                                                  int experts, int top, int softmax,
-                                                                 const float* __restrict__ correction,
+                                                                 const float* __restrict__ correction, RoutePick rule,
                                                                  int* __restrict__ ids, float* __restrict__ weights) {
   ls_dependency_sync();
   const int t = blockIdx.x * ROUTE_WARPS + (threadIdx.x >> 5);
   if (t >= tokens) return;
-  route_token(logits, ld, t, experts, top, softmax, correction, ids, weights);
+  route_token(logits, ld, t, experts, top, softmax, correction, rule, ids, weights);
 }
 
 // plan [0] = tiles, then (expert, first row, rows) per tile; row_token / row_weight per sorted
@@ -188,12 +262,12 @@ __global__ void __launch_bounds__(PLAN_THREADS) plan_kernel(const int* __restric
 // block sorts the pairs.  `real`: the experts that have rows (the first of the `experts` the router scores).
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_plan_kernel(
     const float* __restrict__ logits, int64_t ld, int tokens, int experts, int top, int softmax,
-    const float* __restrict__ correction, int* ids, float* weights, int real, int tile_rows,
+    const float* __restrict__ correction, RoutePick rule, int* ids, float* weights, int real, int tile_rows,
     int* __restrict__ plan, int max_tiles, int* __restrict__ row_token, float* __restrict__ row_weight,
     int* __restrict__ pair_row, int* err) {
   ls_dependency_sync();
   for (int t = threadIdx.x >> 5; t < tokens; t += ROUTE_WARPS)
-    route_token(logits, ld, t, experts, top, softmax, correction, ids, weights);
+    route_token(logits, ld, t, experts, top, softmax, correction, rule, ids, weights);
   __syncthreads();                  // (the block's own writes to ids and weights are visible to it behind the barrier)
   plan_block(ids, weights, tokens * top, top, real, tile_rows, plan, max_tiles, row_token, row_weight, pair_row, err);
 }
@@ -321,33 +395,42 @@ __global__ void __launch_bounds__(256) mix_kernel(const float* __restrict__ y, c
   }
 }
 
+// groups 0: no limit; else equal groups, the kept ones of which hold enough experts
+bool pick_ok(int experts, int top, int groups, int keep) {
+  if (groups == 0) return true;
+  return groups > 0 && groups <= experts && experts % groups == 0 && keep > 0 && keep <= groups &&
+         (long long)keep * (experts / groups) >= top;
+}
+
 }  // namespace
 
 LS_API int ls_experts_tile_rows() { return TILE_M; }
 
 LS_API int ls_experts_route(const float* logits, long long ld, int tokens, int experts, int top, int softmax,
-                            const float* correction, int* ids, float* weights, cudaStream_t stream) {
+                            const float* correction, int groups, int keep, float factor, int* ids, float* weights, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (!pick_ok(experts, top, groups, keep)) return LS_E_SIZE;
   if (experts <= 0 || experts > 32 * MAX_PER_LANE || top <= 0 || top > experts || ld < experts) return LS_E_SIZE;
   LS_COUNT(LS_K_EXPERTS_ROUTE);
   cudaError_t e = ls_launch(route_kernel, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream,
-                            logits, (int64_t)ld, tokens, experts, top, softmax, correction, ids, weights);
+                            logits, (int64_t)ld, tokens, experts, top, softmax, correction, RoutePick{groups, keep, factor}, ids, weights);
   if (e != cudaSuccess) return (int)e;
   return ls_launch_status();
 }
 
 // Both in one launch of one block, for steps of few tokens (the same choices, weights and plan).
 LS_API int ls_experts_route_plan(const float* logits, long long ld, int tokens, int experts, int top, int softmax,
-                                 const float* correction, int* ids, float* weights, int real, int tile_rows, int* plan,
+                                 const float* correction, int groups, int keep, float factor, int* ids, float* weights, int real, int tile_rows, int* plan,
                                  int max_tiles, int* row_token, float* row_weight, int* pair_row, int* err,
                                  cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (!pick_ok(experts, top, groups, keep)) return LS_E_SIZE;
   if (experts <= 0 || experts > 32 * MAX_PER_LANE || top <= 0 || top > experts || ld < experts) return LS_E_SIZE;
   if (real <= 0 || real > experts || max_tiles <= 0 || tile_rows <= 0) return LS_E_SIZE;
   LS_COUNT(LS_K_EXPERTS_ROUTE);
   LS_COUNT(LS_K_EXPERTS_PLAN);
   cudaError_t e = ls_launch(route_plan_kernel, dim3(1), dim3(ROUTE_WARPS * 32), sizeof(int) * 3 * (size_t)real, stream,
-                            logits, (int64_t)ld, tokens, experts, top, softmax, correction, ids, weights, real, tile_rows,
+                            logits, (int64_t)ld, tokens, experts, top, softmax, correction, RoutePick{groups, keep, factor}, ids, weights, real, tile_rows,
                             plan, max_tiles, row_token, row_weight, pair_row, err);
   if (e != cudaSuccess) return (int)e;
   return ls_launch_status();

@@ -14,6 +14,7 @@
 //   2 silu-mul     C[m, n]  = silu(acc_gate) * acc_up   (W holds gate rows [0, N)
 //                                                        and up rows [N, 2N))
 //   4 gelu         C[m, n]  = gelu_tanh(acc)
+//   5 relu squared C[m, n]  = max(acc, 0)^2
 #include "common.cuh"
 
 namespace {
@@ -88,6 +89,8 @@ gemm_nt_kernel(const TA* __restrict__ A, const TW* __restrict__ W, TC* __restric
         *c = ls_from_float<TC>(ls_to_float<TC>(*c) + acc[i][j]);
       } else if (EPI == 4) {
         *c = ls_from_float<TC>(ls_gelu_tanh(acc[i][j]));
+      } else if (EPI == 5) {
+        *c = ls_from_float<TC>(ls_relu_squared(acc[i][j]));
       } else {
         const float g = acc[i][j];
         *c = ls_from_float<TC>(g / (1.0f + expf(-g)) * acu[i][j]);
@@ -216,6 +219,8 @@ gemm_nt_skinny_kernel(const float* __restrict__ A, const float* __restrict__ W, 
         *c = ls_from_float<TC>(ls_to_float<TC>(*c) + acc[i]);
       } else if (EPI == 4) {
         *c = ls_from_float<TC>(ls_gelu_tanh(acc[i]));
+      } else if (EPI == 5) {
+        *c = ls_from_float<TC>(ls_relu_squared(acc[i]));
       } else {
         const float g = acc[i];
         *c = ls_from_float<TC>(g / (1.0f + expf(-g)) * acu[i]);
@@ -374,7 +379,8 @@ gemm_nt_large_kernel(const float* __restrict__ A, const float* __restrict__ W, f
 #pragma unroll
       for (int j = 0; j < WC; ++j) {
         const int n = n0 + (j < 4 ? tx * 4 + j : 64 + tx * 4 + j - 4);
-        if (n < N) crow[n] = EPI == 1 ? crow[n] + acc[i][j] : EPI == 4 ? ls_gelu_tanh(acc[i][j]) : acc[i][j];
+        if (n < N) crow[n] = EPI == 1 ? crow[n] + acc[i][j] : EPI == 4 ? ls_gelu_tanh(acc[i][j])
+                         : EPI == 5 ? ls_relu_squared(acc[i][j]) : acc[i][j];
       }
     }
   }
@@ -431,6 +437,9 @@ int launch(const void* A, const void* W, void* C, int M, int N, int K, int64_t l
     case 4:
       LS_COUNT(LS_K_GEMM_SIMT), ls_launch(gemm_nt_kernel<TA, TW, TC, 4>, grid, 256, 0, stream, (const TA*)A, (const TW*)W, (TC*)C, M, N, K, lda, ldw, ldc);
       break;
+    case 5:
+      LS_COUNT(LS_K_GEMM_SIMT), ls_launch(gemm_nt_kernel<TA, TW, TC, 5>, grid, 256, 0, stream, (const TA*)A, (const TW*)W, (TC*)C, M, N, K, lda, ldw, ldc);
+      break;
     default:
       return LS_E_SIZE;
   }
@@ -455,6 +464,7 @@ LS_API int ls_gemm_nt_simt(const void* A, const void* W, void* C, int a_dtype, i
     if (epilogue == 1) return launch_skinny<1>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     if (epilogue == 2) return launch_skinny<2>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     if (epilogue == 4) return launch_skinny<4>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
+    if (epilogue == 5) return launch_skinny<5>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     return LS_E_SIZE;
   }
   // float32 rows that can be fetched 16 bytes at a time, more than a few of them
@@ -466,6 +476,7 @@ LS_API int ls_gemm_nt_simt(const void* A, const void* W, void* C, int a_dtype, i
     if (epilogue == 1) return launch_large<1>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     if (epilogue == 2) return launch_large<2>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     if (epilogue == 4) return launch_large<4>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
+    if (epilogue == 5) return launch_large<5>(a, w, (float*)C, M, N, K, lda, ldw, ldc, stream);
     return LS_E_SIZE;
   }
   if (a_dtype == LS_F32 && c_dtype == LS_F32)

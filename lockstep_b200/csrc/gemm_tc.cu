@@ -95,9 +95,15 @@ __device__ __forceinline__ float gelu_tanh(float a) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z2 * -1.4426950408889634f));
   return __fdividef(a, 1.0f + e);
 }
-// what an epilogue that stores one sum an output writes (EPI 4: its gelu)
+// what an epilogue that stores one sum an output writes (EPI 4: its gelu, EPI 5: the square of its relu)
 template <int EPI>
-__device__ __forceinline__ float finished(float a) { return EPI == 4 ? gelu_tanh(a) : a; }
+__device__ __forceinline__ float finished(float a) {
+  if (EPI == 5) {
+    const float r = fmaxf(a, 0.f);
+    return r * r;
+  }
+  return EPI == 4 ? gelu_tanh(a) : a;
+}
 
 __host__ __device__ constexpr int tmem_cols(int n) { return n <= 32 ? 32 : n <= 64 ? 64 : n <= 128 ? 128 : n <= 256 ? 256 : 512; }
 
@@ -114,7 +120,7 @@ struct Shape {
 
 template <int EPI, typename TC>
 __device__ __forceinline__ void epilogue_store(TC* c, float a, float up) {
-  if (EPI == 0 || EPI == 4) {
+  if (EPI == 0 || EPI >= 4) {
     *c = ls_from_float<TC>(finished<EPI>(a));
   } else if (EPI == 1) {
     *c = ls_from_float<TC>(ls_to_float<TC>(*c) + a);
@@ -1071,7 +1077,7 @@ gemm_tc_walk_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
               if (t < T) {
                 TC* c = C + (int64_t)t * ldc + n;
                 const float a = sum[c0 + j];
-                if (EPI == 0 || EPI == 4) *c = ls_from_float<TC>(finished<EPI>(a));
+                if (EPI == 0 || EPI >= 4) *c = ls_from_float<TC>(finished<EPI>(a));
                 else if (EPI == 1) *c = ls_from_float<TC>(old[j] + a);
                 else *c = ls_from_float<TC>(silu_mul(a, sum[TOK + c0 + j]));
               }
@@ -1761,6 +1767,9 @@ int run_rows(const void* X, const void* W, void* C, int c_dtype, int T, int N, i
   if (epilogue == 4 && c_dtype == LS_BF16)
     return wide ? launch_rows_as<4, 256, bf16>(mw, mx, C, T, N, K, ldc, plan, err, stream)
                 : launch_rows_as<4, 128, bf16>(mw, mx, C, T, N, K, ldc, plan, err, stream);
+  if (epilogue == 5 && c_dtype == LS_BF16)
+    return wide ? launch_rows_as<5, 256, bf16>(mw, mx, C, T, N, K, ldc, plan, err, stream)
+                : launch_rows_as<5, 128, bf16>(mw, mx, C, T, N, K, ldc, plan, err, stream);
   if (epilogue == 0 && c_dtype == LS_F32)
     return wide ? launch_rows_as<0, 256, float>(mw, mx, C, T, N, K, ldc, plan, err, stream)
                 : launch_rows_as<0, 128, float>(mw, mx, C, T, N, K, ldc, plan, err, stream);
@@ -1818,13 +1827,15 @@ int dispatch(const CUtensorMap& mw, const CUtensorMap& mx, const NormArgs* norm,
     return launch<BN, 3, bf16>(mw, mx, norm, heads, C, T, N, K, ldc, plan, err, stream);
   if (epilogue == 4 && c_dtype == LS_BF16)
     return launch<BN, 4, bf16>(mw, mx, norm, heads, C, T, N, K, ldc, plan, err, stream);
+  if (epilogue == 5 && c_dtype == LS_BF16)
+    return launch<BN, 5, bf16>(mw, mx, norm, heads, C, T, N, K, ldc, plan, err, stream);
   return LS_E_DTYPE;
 }
 
 int run(const void* X, const NormArgs* norm, const LsQkvStore* heads, const void* W, void* C, int c_dtype, int T,
         int N, int K, int64_t ldx, int64_t ldw, int64_t ldc, int epilogue, int* err, cudaStream_t stream) {
   if (T <= 0 || N <= 0) return 0;
-  if (K <= 0 || epilogue < 0 || epilogue > 4 || (epilogue == 3) != (heads != nullptr)) return LS_E_SIZE;
+  if (K <= 0 || epilogue < 0 || epilogue > 5 || (epilogue == 3) != (heads != nullptr)) return LS_E_SIZE;
   if ((K % 8) || (ldw % 8)) return LS_E_ALIGN;     // 16-byte row pitch
   if ((uintptr_t)W & 15) return LS_E_ALIGN;
   if ((N + BM - 1) / BM > 2147483647 / 2 || (T + 15) / 16 > 65535) return LS_E_SIZE;

@@ -6,15 +6,22 @@
 //   - biases of the three projections, added here (in float32) rather than in the product;
 //   - a query temperature: the query of position p times 1 + coef ln(floor((p + 1) / every) + 1);
 //   - rotation of neighbouring pairs (2i, 2i + 1) instead of (i, i + rot_dim / 2);
-//   - values mixed with another projection's values of the same token: v <- (1 - mix) v + mix other.
+//   - values mixed with another projection's values of the same token: v <- (1 - mix) v + mix other;
+//   - several maps a head (differential attention): q and k have `maps` sub-heads of size d per head, each normed
+//     (and rotated) by itself.  A key head's sub-heads lie side by side in its one row of D elements; a query
+//     sub-head is a query head of its own whose d elements lie where its map's key lies, zeros elsewhere, so that
+//     its score is its own map's alone and all maps share the one cached value.
+// And what follows the attention of two maps: map_difference, out = rms(a1 - lambda a2) factor sigmoid(gate_h) over a
+// head's dv values, from the attention's rows or, for decoded tokens, from the partials of their splits.
 // Queries go to q_out [tokens, nq * D], keys and values into the cache pages
-// [num_pages, 2, nkv, page_size, D]; D >= max(d, dv) is the one head size the attention
+// [num_pages, 2, nkv, page_size, D]; D >= max(maps d, dv) is the one head size the attention
 // kernels then work with, and the elements past d (dv) are written as zeros: a zero in a
 // query or key adds nothing to a score, a zero value column gives a zero output column.
 // One block per token.  Sums of squares are taken in float32 in a fixed order (a thread's
 // elements ascending, lanes by xor-tree, warps ascending), so a token's bits do not depend
 // on the batch.  Rotation: halves or neighbouring pairs of the first rot_dim elements of each head,
 // products and sums rounded one by one as in rope.cuh.
+#include "attention_fold.cuh"
 #include "common.cuh"
 
 namespace {
@@ -22,7 +29,7 @@ namespace {
 constexpr int THREADS = 256;
 
 struct WideArgs {
-  const void* qkv;          // [tokens, ld]: q (nq*d), then k (nkv*d) and v (nkv*dv) if has_kv
+  const void* qkv;          // [tokens, ld]: q (nq*d), then k (nkv*maps*d) and v (nkv*dv) if has_kv; nq counts sub-heads
   void* q_out;
   void* pages;
   const void* q_gain;       // scope 2: [nq*d]; scope 1: [d]; null: no norm
@@ -45,6 +52,7 @@ struct WideArgs {
   const void* v_other;      // null, or [tokens, v_other_ld]: values to mix into this layer's
   int64_t v_other_ld;
   const float* v_mix;       // one number
+  int maps;                 // sub-heads of a head (1: none)
 };
 
 __device__ __forceinline__ float gain_at(const void* g, int bf16, int i) {
@@ -71,8 +79,9 @@ __device__ float block_sumsq(const WideArgs& a, const T* src, int col0, int n, f
 }
 
 // One projection (q or k) of one token: heads of size d at src, normed, rotated, written as
-// heads of size D at dst(head) (the padding as zeros).
-template <typename T, typename Dst>
+// heads of size D at dst(head) (the padding as zeros).  KEYS: `maps` of them share a row of D, side by side;
+// else (queries) each has a row of its own, its elements at its map's place.
+template <typename T, bool KEYS, typename Dst>
 __device__ void finish_heads(const WideArgs& a, const T* src, int col0, int heads, const void* gain, float rstd_whole,
                              const float* cs, const float* sn, float* head_rstd, float factor, Dst dst) {
   const int d = a.d, D = a.D, half = a.rot_dim >> 1;
@@ -90,8 +99,16 @@ __device__ void finish_heads(const WideArgs& a, const T* src, int col0, int head
     }
     __syncthreads();
   }
-  for (int e = threadIdx.x; e < heads * D; e += THREADS) {
-    const int h = e / D, i = e - h * D;
+  const int rows = KEYS ? heads / a.maps : heads;
+  for (int e = threadIdx.x; e < rows * D; e += THREADS) {
+    const int row = e / D, at = e - row * D;
+    int h = row, i = at;                                 // the head and the element of it that lie here
+    if (a.maps > 1) {
+      const int map = at / d;
+      const bool here = map < a.maps && (KEYS || map == row % a.maps);
+      if (KEYS) h = row * a.maps + map;
+      i = here ? at - map * d : d;
+    }
     float out = 0.f;
     if (i < d) {
       auto normed = [&](int j) {
@@ -120,7 +137,7 @@ __device__ void finish_heads(const WideArgs& a, const T* src, int col0, int head
       }
       if (factor != 1.0f) out = __fmul_rn(out, factor);
     }
-    dst(h, i, out);
+    dst(row, at, out);
   }
 }
 
@@ -147,7 +164,7 @@ __global__ void __launch_bounds__(THREADS) qkv_finish_kernel(WideArgs a, int* er
   T* q_dst = reinterpret_cast<T*>(a.q_out) + (int64_t)t * a.nq * a.D;
   const float temperature =
       a.temp_coef != 0.f ? 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1)) : 1.0f;
-  finish_heads<T>(a, row, 0, a.nq, a.q_gain, rstd, cs, sn, head_rstd, temperature,
+  finish_heads<T, false>(a, row, 0, a.nq, a.q_gain, rstd, cs, sn, head_rstd, temperature,
                   [&](int h, int i, float v) { q_dst[h * a.D + i] = ls_from_float<T>(v); });
   if (!a.has_kv || !a.write_cache) return;
 
@@ -161,14 +178,14 @@ __global__ void __launch_bounds__(THREADS) qkv_finish_kernel(WideArgs a, int* er
   const int in_page = pos % a.page_size;
   T* pages = reinterpret_cast<T*>(a.pages);
   const T* k_src = row + a.nq * a.d;
-  const T* v_src = k_src + a.nkv * a.d;
+  const T* v_src = k_src + a.nkv * a.maps * a.d;
   float k_rstd = 1.f;
   if (a.scope == 2 && a.k_gain != nullptr) {
     __syncthreads();
-    k_rstd = 1.0f / sqrtf(block_sumsq<T>(a, k_src, a.nq * a.d, a.nkv * a.d, scratch) / (float)(a.nkv * a.d) + a.eps);
+    k_rstd = 1.0f / sqrtf(block_sumsq<T>(a, k_src, a.nq * a.d, a.nkv * a.maps * a.d, scratch) / (float)(a.nkv * a.maps * a.d) + a.eps);
   }
   __syncthreads();          // head_rstd is used again
-  finish_heads<T>(a, k_src, a.nq * a.d, a.nkv, a.k_gain, k_rstd, cs, sn, head_rstd, 1.0f, [&](int h, int i, float v) {
+  finish_heads<T, true>(a, k_src, a.nq * a.d, a.nkv * a.maps, a.k_gain, k_rstd, cs, sn, head_rstd, 1.0f, [&](int h, int i, float v) {
     pages[((((int64_t)page * 2 + 0) * a.nkv + h) * a.page_size + in_page) * a.D + i] = ls_from_float<T>(v);
   });
   const T* other = a.v_other != nullptr ? reinterpret_cast<const T*>(a.v_other) + (int64_t)t * a.v_other_ld : nullptr;
@@ -177,14 +194,126 @@ __global__ void __launch_bounds__(THREADS) qkv_finish_kernel(WideArgs a, int* er
     const int h = e / a.D, i = e - h * a.D;
     float v = 0.f;
     if (i < a.dv) {
-      v = biased_at<T>(a, v_src, (a.nq + a.nkv) * a.d, h * a.dv + i);
+      v = biased_at<T>(a, v_src, (a.nq + a.nkv * a.maps) * a.d, h * a.dv + i);
       if (other != nullptr) v = __fadd_rn(__fmul_rn(1.0f - mix, v), __fmul_rn(mix, ls_to_float<T>(other[h * a.dv + i])));
     }
     pages[((((int64_t)page * 2 + 1) * a.nkv + h) * a.page_size + in_page) * a.D + i] = ls_from_float<T>(v);
   }
 }
 
+// ---------------------------------------------------------------------------------------
+// The difference of two maps: attention heads 2 h and 2 h + 1 are the maps of head h,
+//   out[t, h, :] = u / sqrt(mean(u^2) + eps) * factor * sigmoid(gate[t, h]),  u = a_(2h) - lambda a_(2h+1),
+// over the first dv elements of the attention's heads of D; float32 inside.  The sum of squares: a lane's
+// elements c = lane, lane + 32, ... ascending, the lanes by an xor tree.
+// ---------------------------------------------------------------------------------------
+constexpr int DIFF_WARPS = 8;
+
+template <typename T>
+__device__ __forceinline__ float diff_gate(const T* __restrict__ gate, int64_t gate_ld, int t, int h, float factor) {
+  return gate == nullptr ? factor : factor / (1.0f + expf(-ls_to_float<T>(gate[(int64_t)t * gate_ld + h])));
+}
+
+// rows of the attention's output: a warp per (token, head)
+template <typename T>
+__global__ void __launch_bounds__(DIFF_WARPS * 32)
+map_difference_kernel(const T* __restrict__ attn, const T* __restrict__ gate, int64_t gate_ld, T* __restrict__ out, int tokens,
+                      int H, int D, int dv, float lambda, float factor, float eps) {
+  ls_dependency_sync();
+  const int64_t item = (int64_t)blockIdx.x * DIFF_WARPS + (threadIdx.x >> 5);
+  if (item >= (int64_t)tokens * H) return;
+  const int t = (int)(item / H), h = (int)(item - (int64_t)t * H), lane = threadIdx.x & 31;
+  const T* a1 = attn + ((int64_t)t * 2 * H + 2 * h) * D;
+  const T* a2 = a1 + D;
+  float u[8], ss = 0.f;                                 // dv <= 256
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int c = lane + 32 * j;
+    u[j] = c < dv ? fmaf(-lambda, ls_to_float<T>(a2[c]), ls_to_float<T>(a1[c])) : 0.f;
+    ss = fmaf(u[j], u[j], ss);
+  }
+  ss = ls_warp_sum(ss);
+  const float f = diff_gate<T>(gate, gate_ld, t, h, factor) / sqrtf(ss / (float)dv + eps);
+  T* dst = out + ((int64_t)t * H + h) * dv;
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int c = lane + 32 * j;
+    if (c < dv) dst[c] = ls_from_float<T>(u[j] * f);
+  }
+}
+
+// decoded tokens: a block per (combine item, head) folds both maps' splits first (each map's output is rounded to the
+// engine's type, as the separate fold stores it: the same bits)
+template <typename T>
+__global__ void __launch_bounds__(256)
+map_difference_fold_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, const int* __restrict__ items,
+                           const T* __restrict__ gate, int64_t gate_ld, T* __restrict__ out, int H, int D, int dv, float lambda,
+                           float factor, float eps) {
+  __shared__ float us[256];
+  __shared__ float sum;
+  ls_dependency_sync();
+  const int* it = items + (int64_t)blockIdx.x * 4;
+  const int tok = it[0], first = it[1], stride = it[2], n = it[3];
+  if (n == 0) return;                                   // padding item of a recorded launch
+  const int h = blockIdx.y, tid = threadIdx.x;
+  for (int c = tid; c < dv; c += blockDim.x) {
+    const float a1 = ls_fold_row(part_acc, part_ml, first, stride, n, 2 * H, 2 * h, D, c);
+    const float a2 = ls_fold_row(part_acc, part_ml, first, stride, n, 2 * H, 2 * h + 1, D, c);
+    us[c] = fmaf(-lambda, ls_to_float<T>(ls_from_float<T>(a2)), ls_to_float<T>(ls_from_float<T>(a1)));
+  }
+  __syncthreads();
+  if (tid < 32) {
+    float ss = 0.f;
+    for (int j = 0; j < 8; ++j) {
+      const int c = tid + 32 * j;
+      const float v = c < dv ? us[c] : 0.f;
+      ss = fmaf(v, v, ss);
+    }
+    ss = ls_warp_sum(ss);
+    if (tid == 0) sum = ss;
+  }
+  __syncthreads();
+  const float f = diff_gate<T>(gate, gate_ld, tok, h, factor) / sqrtf(sum / (float)dv + eps);
+  for (int c = tid; c < dv; c += blockDim.x) out[((int64_t)tok * H + h) * dv + c] = ls_from_float<T>(us[c] * f);
+}
+
 }  // namespace
+
+LS_API int ls_map_difference(const void* attn, const void* gate, int64_t gate_ld, void* out, int dtype, int tokens, int H, int D,
+                             int dv, float lambda, float factor, float eps, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (H <= 0 || dv <= 0 || dv > 256 || D < dv || (gate != nullptr && gate_ld < H)) return LS_E_SIZE;
+  const int64_t items = (int64_t)tokens * H;
+  const dim3 grid((unsigned)((items + DIFF_WARPS - 1) / DIFF_WARPS)), block(DIFF_WARPS * 32);
+  LS_COUNT(LS_K_MAP_DIFFERENCE);
+  typedef __nv_bfloat16 bf16;
+  if (dtype == LS_F32)
+    ls_launch(map_difference_kernel<float>, grid, block, 0, stream, (const float*)attn, (const float*)gate, gate_ld, (float*)out,
+              tokens, H, D, dv, lambda, factor, eps);
+  else if (dtype == LS_BF16)
+    ls_launch(map_difference_kernel<bf16>, grid, block, 0, stream, (const bf16*)attn, (const bf16*)gate, gate_ld, (bf16*)out,
+              tokens, H, D, dv, lambda, factor, eps);
+  else return LS_E_DTYPE;
+  return ls_launch_status();
+}
+
+LS_API int ls_map_difference_fold(const float* part_acc, const float* part_ml, const int* items, int n_items, const void* gate,
+                                  int64_t gate_ld, void* out, int dtype, int H, int D, int dv, float lambda, float factor,
+                                  float eps, cudaStream_t stream) {
+  if (n_items <= 0) return 0;
+  if (H <= 0 || H > 65535 || dv <= 0 || dv > 256 || D < dv || (gate != nullptr && gate_ld < H)) return LS_E_SIZE;
+  const dim3 grid(n_items, H), block(dv > 128 ? 256 : dv > 64 ? 128 : 64);
+  LS_COUNT(LS_K_MAP_DIFFERENCE_FOLD);
+  typedef __nv_bfloat16 bf16;
+  if (dtype == LS_F32)
+    ls_launch(map_difference_fold_kernel<float>, grid, block, 0, stream, part_acc, part_ml, items, (const float*)gate, gate_ld,
+              (float*)out, H, D, dv, lambda, factor, eps);
+  else if (dtype == LS_BF16)
+    ls_launch(map_difference_fold_kernel<bf16>, grid, block, 0, stream, part_acc, part_ml, items, (const bf16*)gate, gate_ld,
+              (bf16*)out, H, D, dv, lambda, factor, eps);
+  else return LS_E_DTYPE;
+  return ls_launch_status();
+}
 
 LS_API int ls_qkv_finish(const void* qkv, int64_t ld, void* q_out, void* pages, int dtype, const void* q_gain,
                          const void* k_gain, int gain_dtype, const float* cos_table, const float* sin_table,
@@ -192,18 +321,19 @@ LS_API int ls_qkv_finish(const void* qkv, int64_t ld, void* q_out, void* pages, 
                          int tokens, int nq, int nkv, int d, int dv, int D, int rot_dim, int page_size,
                          int num_pages, int max_positions, float eps, int scope, int has_kv, int write_cache,
                          const void* bias, int bias_dtype, float temp_coef, int temp_every, int interleaved,
-                         const void* v_other, int64_t v_other_ld, const float* v_mix, int* err, cudaStream_t stream) {
+                         const void* v_other, int64_t v_other_ld, const float* v_mix, int maps, int* err, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (nq <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || D < d || D < dv || scope < 0 || scope > 2) return LS_E_SIZE;
+  if (nq <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || maps < 1 || D < (int64_t)maps * d || D < dv || scope < 0 || scope > 2 || nq % maps)
+    return LS_E_SIZE;
   if (rot_dim < 0 || rot_dim > d || (rot_dim & 1)) return LS_E_SIZE;
-  if (scope == 1 && (nq > 256 || nkv > 256)) return LS_E_SIZE;
+  if (scope == 1 && (nq > 256 || (int64_t)nkv * maps > 256)) return LS_E_SIZE;
   if (gain_dtype != LS_F32 && gain_dtype != LS_BF16) return LS_E_DTYPE;
   if (write_cache && (pages == nullptr || page_size <= 0)) return LS_E_SIZE;
   if (temp_coef != 0.f && temp_every <= 0) return LS_E_SIZE;
   if (bias != nullptr && bias_dtype != LS_F32 && bias_dtype != LS_BF16) return LS_E_DTYPE;
   if (v_other != nullptr && (v_mix == nullptr || !has_kv || v_other_ld < (int64_t)nkv * dv)) return LS_E_SIZE;
   WideArgs a;
-  a.interleaved = interleaved; a.v_other = v_other; a.v_other_ld = v_other_ld; a.v_mix = v_mix;
+  a.maps = maps; a.interleaved = interleaved; a.v_other = v_other; a.v_other_ld = v_other_ld; a.v_mix = v_mix;
   a.bias = bias; a.bias_bf16 = bias_dtype == LS_BF16 ? 1 : 0; a.temp_coef = temp_coef; a.temp_every = temp_every > 0 ? temp_every : 1;
   a.qkv = qkv; a.q_out = q_out; a.pages = pages; a.q_gain = q_gain; a.k_gain = k_gain;
   a.cos_table = cos_table; a.sin_table = sin_table; a.positions = positions; a.token_req = token_req;

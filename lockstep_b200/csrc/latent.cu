@@ -12,7 +12,8 @@
 //                   cache write ([c ; k_r ; 0] as the key row, [c ; 0] as the value row) and the
 //                   rotated and padded part of the folded queries.
 //   heads_product:  out[t, h, :] = a[t, h, :] @ w[h]^T for every head at once (the fold of W_uk into
-//                   the queries, and W_uv on the attention's output), an element one chain of fused
+//                   the queries, and W_uv on the attention's output, there optionally times the sigmoid
+//                   of a gate per element), an element one chain of fused
 //                   multiply-adds over ascending k, so a row's bits do not depend on the batch.
 #include "common.cuh"
 
@@ -146,6 +147,7 @@ __global__ void __launch_bounds__(THREADS) latent_finish_kernel(LatentArgs a, in
 
 // ---------------------------------------------------------------------------------------
 // out[t, h * out_hs + n] = sum_k a[t * a_ld + h * a_hs + k] * w[(h * N + n) * K + k]
+// (with a gate: times sigmoid(gate[t * gate_ld + h * N + n]))
 // 64 x 64 outputs a block, 32 of k at a time, 4 x 4 outputs a thread.  Where the rows allow it
 // (`vec`: pitches, head strides and K multiples of a 16-byte piece, aligned bases) both operands
 // come 16 bytes a load, consecutive threads taking consecutive rows, so that the transposed
@@ -179,7 +181,8 @@ __device__ __forceinline__ void hp_load_tile(float (*tile)[HP_T + 4], const T* _
 template <typename T>
 __global__ void __launch_bounds__(256) heads_product_kernel(const T* __restrict__ a, int64_t a_ld, int a_hs,
                                                             const T* __restrict__ w, T* __restrict__ out, int64_t out_ld,
-                                                            int out_hs, int tokens, int N, int K, int vec) {
+                                                            int out_hs, int tokens, int N, int K, int vec,
+                                                            const T* __restrict__ gate, int64_t gate_ld) {
   __shared__ __align__(16) float As[HP_K][HP_T + 4];
   __shared__ __align__(16) float Ws[HP_K][HP_N + 4];
   ls_dependency_sync();
@@ -215,7 +218,10 @@ __global__ void __launch_bounds__(256) heads_product_kernel(const T* __restrict_
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) out[(int64_t)t * out_ld + (int64_t)h * out_hs + n] = ls_from_float<T>(acc[i][j]);
+      if (n >= N) continue;
+      float v = acc[i][j];
+      if (gate != nullptr) v = v / (1.0f + expf(-ls_to_float<T>(gate[(int64_t)t * gate_ld + (int64_t)h * N + n])));
+      out[(int64_t)t * out_ld + (int64_t)h * out_hs + n] = ls_from_float<T>(v);
     }
   }
 }
@@ -254,9 +260,11 @@ LS_API int ls_latent_finish(const void* proj, int64_t ld, const void* kv, int64_
 }
 
 LS_API int ls_heads_product(const void* a, int64_t a_ld, int a_hs, const void* w, void* out, int64_t out_ld, int out_hs,
-                            int dtype, int tokens, int heads, int N, int K, cudaStream_t stream) {
+                            int dtype, int tokens, int heads, int N, int K, const void* gate, int64_t gate_ld,
+                            cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (heads <= 0 || heads > 65535 || N <= 0 || K <= 0) return LS_E_SIZE;
+  if (gate != nullptr && gate_ld < (int64_t)heads * N) return LS_E_SIZE;
   const dim3 grid((tokens + HP_T - 1) / HP_T, (N + HP_N - 1) / HP_N, heads);
   if (grid.y > 65535) return LS_E_SIZE;
   LS_COUNT(LS_K_HEADS_PRODUCT);
@@ -267,10 +275,10 @@ LS_API int ls_heads_product(const void* a, int64_t a_ld, int a_hs, const void* w
   cudaError_t e;
   if (dtype == LS_F32)
     e = ls_launch(heads_product_kernel<float>, grid, dim3(256), 0, stream, (const float*)a, a_ld, a_hs, (const float*)w,
-                  (float*)out, out_ld, out_hs, tokens, N, K, vec);
+                  (float*)out, out_ld, out_hs, tokens, N, K, vec, (const float*)gate, gate_ld);
   else if (dtype == LS_BF16)
     e = ls_launch(heads_product_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)a, a_ld, a_hs,
-                  (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_ld, out_hs, tokens, N, K, vec);
+                  (const __nv_bfloat16*)w, (__nv_bfloat16*)out, out_ld, out_hs, tokens, N, K, vec, (const __nv_bfloat16*)gate, gate_ld);
   else return LS_E_DTYPE;
   if (e != cudaSuccess) return (int)e;
   return ls_launch_status();

@@ -1,9 +1,9 @@
 // Row-wise kernels of designs that norm after a sublayer as well as before it:
-//   - layer norm with a gain and no bias, (x - mean) rsqrt(var + eps) gain, var the mean of the
-//     squared deviations (rows may be gathered through row_index);
+//   - layer norm with a gain and an optional bias, (x - mean) rsqrt(var + eps) gain + bias, var the
+//     mean of the squared deviations (rows may be gathered through row_index);
 //   - the closing kernel of a sublayer: the RMS-normed results of mixers side by side, each with
 //     a gain of its own, summed with one factor; optionally a layer norm of that sum; added to
-//     the residual stream;
+//     the residual stream; optionally the layer norm of the new stream that the next sublayer reads;
 //   - an embedding with a factor on the token's row and a second table indexed by a hash of the
 //     token and the one before it, whose last row serves a sequence's first token;
 //   - float32 rows written into some columns of a wider row of the engine's type; logits times a
@@ -28,12 +28,17 @@ __device__ __forceinline__ float row_sum(float v, float* scratch) {
   return total;
 }
 
-// (x - mean) rsqrt(var + eps) gain over float32 rows.  A thread takes the elements tid, tid + 256, ... of the row and
+// a normed element times its gain, plus the bias where there is one
+__device__ __forceinline__ float scaled(float u, float gain, bool biased, float bias) {
+  return biased ? fmaf(u, gain, bias) : u * gain;
+}
+
+// (x - mean) rsqrt(var + eps) gain (+ bias) over float32 rows.  A thread takes the elements tid, tid + 256, ... of the row and
 // keeps up to eight of them in registers between the passes (rows up to 2,048 wide are read once).
 template <typename TG, typename TO>
 __global__ void __launch_bounds__(ROW_THREADS)
 layernorm_kernel(const float* __restrict__ x, const int* __restrict__ row_index, const TG* __restrict__ gain,
-                 TO* __restrict__ out, int rows, int width, int x_rows, float eps, int* err) {
+                 const TG* __restrict__ bias, TO* __restrict__ out, int rows, int width, int x_rows, float eps, int* err) {
   __shared__ float scratch[32];
   ls_dependency_sync();
   const int r = blockIdx.x, tid = threadIdx.x;
@@ -70,18 +75,23 @@ layernorm_kernel(const float* __restrict__ x, const int* __restrict__ row_index,
 #pragma unroll
   for (int j = 0; j < KEEP; ++j) {
     const int i = tid + j * ROW_THREADS;
-    if (i < width) dst[i] = ls_from_float<TO>((v[j] - mean) * rstd * gain_of<TG>(gain, i));
+    if (i < width)
+      dst[i] = ls_from_float<TO>(scaled((v[j] - mean) * rstd, gain_of<TG>(gain, i), bias != nullptr, bias != nullptr ? gain_of<TG>(bias, i) : 0.f));
   }
   for (int i = tid + KEEP * ROW_THREADS; i < width; i += ROW_THREADS)
-    dst[i] = ls_from_float<TO>((row[i] - mean) * rstd * gain_of<TG>(gain, i));
+    dst[i] = ls_from_float<TO>(scaled((row[i] - mean) * rstd, gain_of<TG>(gain, i), bias != nullptr, bias != nullptr ? gain_of<TG>(bias, i) : 0.f));
 }
 
-// residual += post(scale sum_b rms_b(x_b) gain_b), post = layer norm with post_gain, or nothing.  The merged row
-// lies in shared memory between the passes.
+// residual += post(scale sum_b rms_b(x_b) gain_b), post = layer norm with post_gain (and post_bias), or nothing.  The
+// merged row lies in shared memory between the passes.  With next_gain the layer norm of the new stream, with that gain
+// (and next_bias), is written to next_out: sums and roundings are those of layernorm_kernel on the stored stream.
+template <typename TO>
 __global__ void __launch_bounds__(ROW_THREADS)
 norm_merge_add_kernel(float* __restrict__ residual, const float* __restrict__ branches, int n, int64_t branch_stride,
                       const float* __restrict__ branch_gain, float scale, const float* __restrict__ post_gain,
-                      int rows, int width, float eps_branch, float eps_post) {
+                      const float* __restrict__ post_bias, const float* __restrict__ next_gain,
+                      const float* __restrict__ next_bias, TO* __restrict__ next_out, int rows, int width, float eps_branch,
+                      float eps_post, float eps_next) {
   extern __shared__ float merged[];                 // [width]
   __shared__ float scratch[32];
   ls_dependency_sync();
@@ -116,18 +126,37 @@ norm_merge_add_kernel(float* __restrict__ residual, const float* __restrict__ br
   float* dst = residual + (int64_t)r * width;
   if (post_gain == nullptr) {
 #pragma unroll 4
-    for (int i = tid; i < width; i += ROW_THREADS) dst[i] += merged[i];
-    return;
+    for (int i = tid; i < width; i += ROW_THREADS) dst[i] = merged[i] = dst[i] + merged[i];
+  } else {
+    const float mean = row_sum(s, scratch) / (float)width;
+    float q = 0.f;
+    for (int i = tid; i < width; i += ROW_THREADS) {
+      const float d = merged[i] - mean;
+      q = fmaf(d, d, q);
+    }
+    const float rstd = 1.0f / sqrtf(row_sum(q, scratch) / (float)width + eps_post);
+#pragma unroll 4
+    for (int i = tid; i < width; i += ROW_THREADS) {
+      const float u = (merged[i] - mean) * rstd;
+      dst[i] = merged[i] = dst[i] + scaled(u, post_gain[i], post_bias != nullptr, post_bias != nullptr ? post_bias[i] : 0.f);
+    }
   }
+  if (next_gain == nullptr) return;
+  s = 0.f;
+  for (int i = tid; i < width; i += ROW_THREADS) s += merged[i];
   const float mean = row_sum(s, scratch) / (float)width;
   float q = 0.f;
   for (int i = tid; i < width; i += ROW_THREADS) {
     const float d = merged[i] - mean;
     q = fmaf(d, d, q);
   }
-  const float rstd = 1.0f / sqrtf(row_sum(q, scratch) / (float)width + eps_post);
+  const float rstd = 1.0f / sqrtf(row_sum(q, scratch) / (float)width + eps_next);
+  TO* to = next_out + (int64_t)r * width;
 #pragma unroll 4
-  for (int i = tid; i < width; i += ROW_THREADS) dst[i] += (merged[i] - mean) * rstd * post_gain[i];
+  for (int i = tid; i < width; i += ROW_THREADS) {
+    const float u = (merged[i] - mean) * rstd;
+    to[i] = ls_from_float<TO>(scaled(u, next_gain[i], next_bias != nullptr, next_bias != nullptr ? next_bias[i] : 0.f));
+  }
 }
 
 // out[t] = table[id] factor + pairs[row(previous id, id)]
@@ -286,14 +315,14 @@ inline int blocks_for(int64_t n) { return (int)((n + 255) / 256 < 148 * 16 ? (n 
 
 }  // namespace
 
-LS_API int ls_layernorm(const float* x, const int* row_index, const void* gain, int gain_dtype, void* out, int out_dtype,
+LS_API int ls_layernorm(const float* x, const int* row_index, const void* gain, const void* bias, int gain_dtype, void* out, int out_dtype,
                         int rows, int width, int x_rows, float eps, int* err, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (width <= 0) return LS_E_SIZE;
   const dim3 grid(rows), block(ROW_THREADS);
   LS_COUNT(LS_K_LAYERNORM);
 #define LS_LN(TG, TO) \
-  ls_launch(layernorm_kernel<TG, TO>, grid, block, 0, stream, x, row_index, (const TG*)gain, (TO*)out, rows, width, x_rows, eps, err)
+  ls_launch(layernorm_kernel<TG, TO>, grid, block, 0, stream, x, row_index, (const TG*)gain, (const TG*)bias, (TO*)out, rows, width, x_rows, eps, err)
   if (gain_dtype == LS_F32 && out_dtype == LS_F32) LS_LN(float, float);
   else if (gain_dtype == LS_F32 && out_dtype == LS_BF16) LS_LN(float, __nv_bfloat16);
   else if (gain_dtype == LS_BF16 && out_dtype == LS_BF16) LS_LN(__nv_bfloat16, __nv_bfloat16);
@@ -304,21 +333,30 @@ LS_API int ls_layernorm(const float* x, const int* row_index, const void* gain, 
 }
 
 LS_API int ls_norm_merge_add(float* residual, const float* branches, int n, long long branch_stride, const float* branch_gain,
-                             float scale, const float* post_gain, int rows, int width, float eps_branch, float eps_post,
-                             cudaStream_t stream) {
+                             float scale, const float* post_gain, const float* post_bias, const float* next_gain,
+                             const float* next_bias, void* next_out, int next_dtype, int rows, int width, float eps_branch,
+                             float eps_post, float eps_next, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (width <= 0 || n < 1 || n > 4) return LS_E_SIZE;
   const size_t smem = sizeof(float) * (size_t)width;
   if (smem > 200 * 1024) return LS_E_SMEM;
   static size_t configured = 48 * 1024;
+  if (next_gain != nullptr && (next_out == nullptr || (next_dtype != LS_F32 && next_dtype != LS_BF16))) return LS_E_DTYPE;
   if (smem > configured) {
-    if (cudaFuncSetAttribute(norm_merge_add_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(norm_merge_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+        cudaFuncSetAttribute(norm_merge_add_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return LS_E_SMEM;
     configured = smem;
   }
-  LS_COUNT(LS_K_NORM_MERGE_ADD);
-  ls_launch(norm_merge_add_kernel, dim3(rows), dim3(ROW_THREADS), smem, stream, residual, branches,
-            n, (int64_t)branch_stride, branch_gain, scale, post_gain, rows, width, eps_branch, eps_post);
+  if (next_gain != nullptr) LS_COUNT(LS_K_NORM_MERGE_NORM);
+  else LS_COUNT(LS_K_NORM_MERGE_ADD);
+#define LS_NM(TO)                                                                                                       \
+  ls_launch(norm_merge_add_kernel<TO>, dim3(rows), dim3(ROW_THREADS), smem, stream, residual, branches, n,              \
+            (int64_t)branch_stride, branch_gain, scale, post_gain, post_bias, next_gain, next_bias, (TO*)next_out, rows, \
+            width, eps_branch, eps_post, eps_next)
+  if (next_gain == nullptr || next_dtype == LS_F32) LS_NM(float);
+  else LS_NM(__nv_bfloat16);
+#undef LS_NM
   return ls_launch_status();
 }
 

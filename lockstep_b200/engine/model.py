@@ -27,6 +27,13 @@ class Model:
         self.head = build_part("head", spec.head, runtime)
         self.tied_head = bool(getattr(self.head, "tied", False))
         self.injection = build_part("injection", spec.injection, runtime) if spec.injection is not None else None
+        # every layer runs once and nothing happens to the stream in between: a layer may then do, with its last
+        # kernel, what the next one would begin with
+        runs = spec.schedule
+        if len({run.layer for run in runs}) == len(runs) and not any(run.inject or run.add_embedding for run in runs):
+            for run, after in zip(runs, runs[1:]):
+                if hasattr(self.blocks[run.layer], "follow_with"):
+                    self.blocks[run.layer].follow_with(self.blocks[after.layer])
         # an embedding that keeps something per request (the token before a portion) has a cache entry of its own,
         # after the schedule's
         need = getattr(self.embedding, "cache_need", lambda: None)()

@@ -19,7 +19,7 @@ from .csrc import build as _build
 F32, BF16 = 0, 1
 _DTYPE_CODE = {torch.float32: F32, torch.bfloat16: BF16}
 
-EPILOGUE_STORE, EPILOGUE_RESIDUAL, EPILOGUE_SILU_MUL, EPILOGUE_GELU = 0, 1, 2, 4
+EPILOGUE_STORE, EPILOGUE_RESIDUAL, EPILOGUE_SILU_MUL, EPILOGUE_GELU, EPILOGUE_RELU2 = 0, 1, 2, 4, 5
 FEW_TOKENS = 32      # up to here a product runs in the few-token kernel, which can also finish q/k/v heads
 
 _REFUSALS = {
@@ -53,9 +53,9 @@ _SIGNATURES = {
                          ctypes.c_longlong, c_void_p, c_void_p],
         "ls_clamped_glu": [c_void_p, ctypes.c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_float,
                            c_void_p, c_void_p, c_int, c_float, c_int, c_void_p],
-        "ls_layernorm": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
-        "ls_norm_merge_add": [c_void_p, c_void_p, c_int, ctypes.c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_float,
-                              c_float, c_void_p],
+        "ls_layernorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
+        "ls_norm_merge_add": [c_void_p, c_void_p, c_int, ctypes.c_longlong, c_void_p, c_float, c_void_p, c_void_p, c_void_p,
+                              c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p],
         "ls_pair_embed": [c_void_p, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                           c_int, c_int, ctypes.c_longlong, ctypes.c_longlong, c_float, c_void_p, c_void_p],
         "ls_rows_cast": [c_void_p, c_void_p, c_int, ctypes.c_longlong, c_int, ctypes.c_longlong, c_void_p],
@@ -113,12 +113,16 @@ _SIGNATURES["seq"] = {
     "ls_qkv_finish": [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                       c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                       c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_int, c_float, c_int, c_int, c_void_p,
-                      c_int64, c_void_p, c_void_p, c_void_p],
+                      c_int64, c_void_p, c_int, c_void_p, c_void_p],
+    "ls_map_difference": [c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float,
+                          c_void_p],
+    "ls_map_difference_fold": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int,
+                               c_float, c_float, c_float, c_void_p],
     "ls_latent_finish": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                          c_int, c_float, c_void_p, c_void_p, c_void_p],
     "ls_heads_product": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
-                         c_void_p],
+                         c_void_p, c_int64, c_void_p],
     "ls_sigmoid_power_decay": [c_void_p, c_void_p, ctypes.c_longlong, c_int, c_float, c_void_p],
     "ls_find_portions": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p],
     "ls_delta_prep": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p,
@@ -140,12 +144,12 @@ _SIGNATURES["seq"] = {
                          c_float, c_int64, c_int, c_void_p],
     "ls_tanh_rows": [c_void_p, c_int, ctypes.c_longlong, c_void_p],
     "ls_experts_tile_rows": [],
-    "ls_experts_route": [c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+    "ls_experts_route": [c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p],
     "ls_experts_mix": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                        ctypes.c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "ls_experts_plan": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                         c_void_p, c_void_p],
-    "ls_experts_route_plan": [c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
+    "ls_experts_route_plan": [c_void_p, ctypes.c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_int,
                               c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
     "ls_experts_tc_tile_rows": [],
     "ls_experts_gather": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
@@ -447,30 +451,42 @@ def weighted_sum(residual, branches, scales, bias=None) -> None:
                                      _opt(bias, "bias", torch.float32), residual.shape[-1], _stream()), "weighted_sum")
 
 
-def layernorm(x, gain, out, eps: float, err, row_index=None) -> None:
-    """out = (x - mean) rsqrt(var + eps) gain over float32 rows of ``x`` (all, or those ``row_index`` names)."""
+def layernorm(x, gain, out, eps: float, err, row_index=None, bias=None) -> None:
+    """out = (x - mean) rsqrt(var + eps) gain (+ bias) over float32 rows of ``x`` (all, or those ``row_index`` names)."""
     rows, width = out.shape
     if x.shape[1] != width or gain.numel() != width or (row_index is None and x.shape[0] != rows) \
             or (row_index is not None and row_index.numel() != rows):
         raise KernelError("layernorm: shapes do not agree")
+    if bias is not None and (bias.numel() != width or bias.dtype != gain.dtype):
+        raise KernelError("layernorm: the bias does not match the gain")
     _check(library().ls_layernorm(
-        _dev(x, "x", torch.float32), _opt(row_index, "row_index", torch.int32), _dev(gain, "gain"), _code(gain),
-        _dev(out, "out"), _code(out), rows, width, x.shape[0], float(eps), _dev(err, "err", torch.int32), _stream()), "layernorm")
+        _dev(x, "x", torch.float32), _opt(row_index, "row_index", torch.int32), _dev(gain, "gain"), _opt(bias, "bias"),
+        _code(gain), _dev(out, "out"), _code(out), rows, width, x.shape[0], float(eps), _dev(err, "err", torch.int32), _stream()),
+        "layernorm")
 
 
-def norm_merge_add(residual, branches, branch_gain, scale: float, post_gain, eps_branch: float, eps_post: float) -> None:
+def norm_merge_add(residual, branches, branch_gain, scale: float, post_gain, eps_branch: float, eps_post: float,
+                   post_bias=None, follow=None) -> None:
     """residual += post(scale sum_b rms(branches[b]) branch_gain[b]): ``branches`` float32 [n, rows, width]; with
     ``branch_gain`` (float32 [n, width]) every branch is divided by its root mean square and multiplied by its gain,
     without it the branches are summed as they are; ``post_gain`` (float32 [width]): the sum goes through a layer norm
-    with this gain before it is added."""
+    with this gain (and ``post_bias``) before it is added.  ``follow`` = (gain, bias or None, eps, out): the layer norm
+    of the new stream is written to ``out`` [rows, width] besides, with the bits ``layernorm`` gives (gain float32)."""
     n, rows, width = branches.shape
     if tuple(residual.shape) != (rows, width) or (branch_gain is not None and tuple(branch_gain.shape) != (n, width)) \
             or (post_gain is not None and post_gain.numel() != width):
         raise KernelError("norm_merge_add: shapes do not agree")
+    next_gain, next_bias, eps_next, next_out = follow if follow is not None else (None, None, 0.0, None)
+    if (post_bias is not None and (post_gain is None or post_bias.numel() != width)) \
+            or (next_bias is not None and next_bias.numel() != width) \
+            or (follow is not None and (next_gain.numel() != width or tuple(next_out.shape) != (rows, width))):
+        raise KernelError("norm_merge_add: a bias or the norm that follows does not match")
     _check(library().ls_norm_merge_add(
         _dev(residual, "residual", torch.float32), _dev(branches, "branches", torch.float32), n, rows * width,
         _opt(branch_gain, "branch_gain", torch.float32), float(scale), _opt(post_gain, "post_gain", torch.float32),
-        rows, width, float(eps_branch), float(eps_post), _stream()), "norm_merge_add")
+        _opt(post_bias, "post_bias", torch.float32), _opt(next_gain, "next_gain", torch.float32),
+        _opt(next_bias, "next_bias", torch.float32), _opt(next_out, "next_out"), _code(next_out) if next_out is not None else F32,
+        rows, width, float(eps_branch), float(eps_post), float(eps_next), _stream()), "norm_merge_add")
 
 
 def pair_embed(ids, token_slot, carried, table, pairs, out, factor: float, mul_prev: int, mul_cur: int, err) -> None:
@@ -806,24 +822,26 @@ RULE_DELTA, RULE_WKV, RULE_GLA, RULE_DELTA_HEAD, RULE_MLSTM = 0, 1, 2, 3, 4
 def qkv_finish(qkv, q_out, pages, q_gain, k_gain, cos, sin, positions, token_req, block_table, nq: int, nkv: int,
                d: int, dv: int, pad: int, rot_dim: int, eps: float, whole_projection: bool, has_kv: bool,
                write_cache: bool, err, bias=None, q_temp=None, interleaved: bool = False, v_other=None,
-               v_mix=None) -> None:
-    """Finishes a projection ``qkv`` [tokens, nq*d (+ nkv*d + nkv*dv)]: RMSNorm of q and of k (over
+               v_mix=None, maps: int = 1) -> None:
+    """Finishes a projection ``qkv`` [tokens, nq*d (+ nkv*d + nkv*dv)] (which may be columns of a wider tensor): RMSNorm of q and of k (over
     the whole projection, or per head), rotation of the first ``rot_dim`` elements of each head,
     queries to ``q_out`` [tokens, nq*pad] and keys and values into ``pages``
     [num_pages, 2, nkv, page_size, pad], padded with zeros (csrc/heads_wide.cu).  ``bias`` (one
     element per column of ``qkv``, or None) is added first; ``q_temp`` = (coef, every): the query at
     position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  ``interleaved``: neighbouring elements
     are rotated as pairs instead of the halves.  ``v_other`` ([tokens, nkv*dv], possibly columns of a wider tensor)
-    and ``v_mix`` (one float32): v <- (1 - v_mix) v + v_mix v_other before the values are written."""
+    and ``v_mix`` (one float32): v <- (1 - v_mix) v + v_mix v_other before the values are written.  ``maps``: every head has
+    that many sub-heads of ``d`` elements (``nq`` counts the queries', the keys have nkv * maps): a key head's lie side by
+    side in its row of ``pad`` elements, a query's where its map's key lies, with zeros around it."""
     tokens = qkv.shape[0]
-    cols = nq * d + (nkv * (d + dv) if has_kv else 0)
-    if qkv.shape[1] != cols or q_out.shape != (tokens, nq * pad) or q_out.dtype != qkv.dtype:
+    cols = nq * d + (nkv * (maps * d + dv) if has_kv else 0)
+    if maps < 1 or nq % maps or qkv.shape[1] != cols or q_out.shape != (tokens, nq * pad) or q_out.dtype != qkv.dtype:
         raise KernelError("qkv_finish: shapes do not agree")
     gains = [g for g in (q_gain, k_gain) if g is not None]
     if any(g.dtype != gains[0].dtype for g in gains):
         raise KernelError("qkv_finish: gains of two element types")
     want_q = nq * d if whole_projection else d
-    want_k = nkv * d if whole_projection else d
+    want_k = nkv * maps * d if whole_projection else d
     if (q_gain is not None and q_gain.numel() != want_q) or (k_gain is not None and k_gain.numel() != want_k):
         raise KernelError("qkv_finish: gains do not match the projection")
     if write_cache:
@@ -842,8 +860,9 @@ def qkv_finish(qkv, q_out, pages, q_gain, k_gain, cos, sin, positions, token_req
         if v_other.dtype != qkv.dtype or tuple(v_other.shape) != (tokens, nkv * dv) or v_mix is None or v_mix.numel() != 1:
             raise KernelError("qkv_finish: the values to mix in do not match")
         vp, v_ld = _rows(v_other, "v_other")
+    qp, q_ld = _rows(qkv, "qkv")
     _check(library("seq").ls_qkv_finish(
-        _dev(qkv, "qkv"), qkv.shape[1], _dev(q_out, "q_out"), _opt(pages if write_cache else None, "pages"),
+        qp, q_ld, _dev(q_out, "q_out"), _opt(pages if write_cache else None, "pages"),
         _code(qkv), _opt(q_gain, "q_gain"), _opt(k_gain, "k_gain"), _code(gains[0]) if gains else F32,
         _opt(cos if rot_dim else None, "cos", torch.float32), _opt(sin if rot_dim else None, "sin", torch.float32),
         _dev(positions, "positions", torch.int32), _dev(token_req, "token_req", torch.int32),
@@ -851,7 +870,7 @@ def qkv_finish(qkv, q_out, pages, q_gain, k_gain, cos, sin, positions, token_req
         page_size, num_pages, cos.shape[0] if rot_dim else 0, float(eps), 2 if whole_projection else 1,
         1 if has_kv else 0, 1 if write_cache else 0, _opt(bias, "bias"), _code(bias) if bias is not None else F32,
         coef, every, 1 if interleaved else 0, vp, v_ld, _opt(v_mix if vp else None, "v_mix", torch.float32),
-        _dev(err, "err", torch.int32), _stream()), "qkv_finish")
+        int(maps), _dev(err, "err", torch.int32), _stream()), "qkv_finish")
 
 
 def latent_finish(proj, q_out, pages, gain, cos, sin, positions, token_req, block_table, heads: int, d: int, dr: int,
@@ -891,9 +910,43 @@ def latent_finish(proj, q_out, pages, gain, cos, sin, positions, token_req, bloc
         _dev(err, "err", torch.int32), _stream()), "latent_finish")
 
 
-def heads_product(a, a_head_stride: int, w, out, out_head_stride: int) -> None:
+def map_difference(attn, gate, out, heads: int, dv: int, lam: float, factor: float, eps: float) -> None:
+    """out[t, h] = u / sqrt(mean(u^2) + eps) factor sigmoid(gate[t, h]) with u = a1 - lam a2 over the first ``dv`` elements
+    of attention heads 2 h and 2 h + 1 of ``attn`` [tokens, 2 heads D]; ``gate`` [tokens, heads] (columns of a wider tensor
+    are fine) or None; out [tokens, heads dv]; one element type (csrc/heads_wide.cu)."""
+    tokens = attn.shape[0]
+    gp, g_ld = _map_difference_gate(gate, out, tokens, heads, dv)
+    if attn.shape[1] % (2 * heads) or attn.dtype != out.dtype:
+        raise KernelError("map_difference: the attention's rows do not match")
+    _check(library("seq").ls_map_difference(
+        _dev(attn, "attn"), gp, g_ld, _dev(out, "out"), _code(out), tokens, heads, attn.shape[1] // (2 * heads), dv, float(lam),
+        float(factor), float(eps), _stream()), "map_difference")
+
+
+def map_difference_fold(part_acc, part_ml, items, n_items: int, gate, out, heads: int, dv: int, lam: float, factor: float,
+                        eps: float) -> None:
+    """``attention_combine`` of the items' tokens and ``map_difference`` of their rows in one kernel (the same bits);
+    ``part_acc`` float32 [slots, 2 heads, D]; rows of ``out`` that no item names are left alone."""
+    gp, g_ld = _map_difference_gate(gate, out, out.shape[0], heads, dv)
+    if part_acc.dim() != 3 or part_acc.shape[1] != 2 * heads:
+        raise KernelError("map_difference_fold: the partials do not match")
+    _check(library("seq").ls_map_difference_fold(
+        _dev(part_acc, "part_acc", torch.float32), _dev(part_ml, "part_ml", torch.float32), _dev(items, "items", torch.int32),
+        n_items, gp, g_ld, _dev(out, "out"), _code(out), heads, part_acc.shape[2], dv, float(lam), float(factor), float(eps),
+        _stream()), "map_difference_fold")
+
+
+def _map_difference_gate(gate, out, tokens: int, heads: int, dv: int) -> tuple[int, int]:
+    if tuple(out.shape) != (tokens, heads * dv) or (gate is not None and (tuple(gate.shape) != (tokens, heads)
+                                                                          or gate.dtype != out.dtype)):
+        raise KernelError("map_difference: the gate or the output does not match")
+    return _rows(gate, "gate") if gate is not None else (0, 0)
+
+
+def heads_product(a, a_head_stride: int, w, out, out_head_stride: int, gate=None) -> None:
     """out[t, h out_head_stride + n] = sum_k a[t, h a_head_stride + k] w[h, n, k] for every head h at once:
-    ``a`` and ``out`` are [tokens, columns] (views of some columns of wider tensors are fine), ``w`` [heads, n, k]."""
+    ``a`` and ``out`` are [tokens, columns] (views of some columns of wider tensors are fine), ``w`` [heads, n, k].
+    ``gate`` [tokens, heads n]: every sum is multiplied by the sigmoid of its element before it is rounded."""
     heads, n, k = w.shape
     ap, a_ld = _rows(a, "a")
     op, o_ld = _rows(out, "out")
@@ -901,8 +954,13 @@ def heads_product(a, a_head_stride: int, w, out, out_head_stride: int) -> None:
         raise KernelError("heads_product: shapes or types do not agree")
     if (heads - 1) * a_head_stride + k > a.shape[1] or (heads - 1) * out_head_stride + n > out.shape[1]:
         raise KernelError("heads_product: the heads do not fit the rows")
+    gp, g_ld = (0, 0)
+    if gate is not None:
+        if tuple(gate.shape) != (a.shape[0], heads * n) or gate.dtype != w.dtype:
+            raise KernelError("heads_product: the gate does not match")
+        gp, g_ld = _rows(gate, "gate")
     _check(library("seq").ls_heads_product(ap, a_ld, a_head_stride, _dev(w, "w"), op, o_ld, out_head_stride, _code(w),
-                                           a.shape[0], heads, n, k, _stream()), "heads_product")
+                                           a.shape[0], heads, n, k, gp, g_ld, _stream()), "heads_product")
 
 
 def sigmoid_power_decay(z, bias, tau: float) -> None:
@@ -1070,10 +1128,12 @@ def experts_tile_rows(tensor_cores: bool = False) -> int:
 
 
 def experts_route(logits, top: int, ids, weights, experts: int | None = None, softmax: bool = False,
-                  correction=None) -> None:
+                  correction=None, groups: int = 0, keep: int = 0, factor: float = 0.0) -> None:
     """The ``top`` experts of every token and their weights, from float32 ``logits`` [tokens, >= experts] (the
     first ``experts`` columns; default all; a view of some columns of a wider tensor is fine).  The weight is the sigmoid of the logit, or with ``softmax`` the
-    softmax over the experts; ``correction`` (float32 [experts]) is added to it for the choice alone."""
+    softmax over the experts; ``correction`` (float32 [experts]) is added to it for the choice alone.  ``groups`` and ``keep``: only
+    experts of the ``keep`` best of ``groups`` equal runs of neighbours can be chosen, a run's score the sum of its two largest
+    choice scores; ``factor``: the weights are divided by (their sum + 1e-20) and multiplied by it (0: they stay)."""
     tokens = logits.shape[0]
     experts = logits.shape[1] if experts is None else int(experts)
     if correction is not None and correction.numel() != experts:
@@ -1082,8 +1142,8 @@ def experts_route(logits, top: int, ids, weights, experts: int | None = None, so
         raise KernelError("experts_route: logits must be float32")
     lp, l_ld = _rows(logits, "logits")
     _check(library("seq").ls_experts_route(lp, l_ld, tokens, experts, top,
-                                           int(softmax), _opt(correction, "correction", torch.float32),
-                                           _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32),
+                                           int(softmax), _opt(correction, "correction", torch.float32), int(groups), int(keep),
+                                           float(factor), _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32),
                                            _stream()), "experts_route")
 
 
@@ -1119,7 +1179,8 @@ def experts_plan(ids, weights, experts: int, tile_rows: int, plan, max_tiles: in
 
 
 def experts_route_plan(logits, top: int, ids, weights, experts: int, softmax: bool, correction, real: int, tile_rows: int,
-                       plan, max_tiles: int, row_token, row_weight, pair_row, err) -> None:
+                       plan, max_tiles: int, row_token, row_weight, pair_row, err, groups: int = 0, keep: int = 0,
+                       factor: float = 0.0) -> None:
     """``experts_route`` and ``experts_plan`` (over the first ``real`` experts) in one launch of one block, for steps
     of few tokens: the same choices, weights and plan."""
     tokens = logits.shape[0]
@@ -1128,7 +1189,7 @@ def experts_route_plan(logits, top: int, ids, weights, experts: int, softmax: bo
     lp, l_ld = _rows(logits, "logits")
     _check(library("seq").ls_experts_route_plan(
         lp, l_ld, tokens, experts, top, int(softmax), _opt(correction, "correction", torch.float32),
-        _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32), real, tile_rows,
+        int(groups), int(keep), float(factor), _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32), real, tile_rows,
         _dev(plan, "plan", torch.int32), max_tiles, _dev(row_token, "row_token", torch.int32),
         _dev(row_weight, "row_weight", torch.float32), _dev(pair_row, "pair_row", torch.int32),
         _dev(err, "err", torch.int32), _stream()), "experts_route_plan")

@@ -44,7 +44,8 @@ class CacheNeed:
 
     kind "paged_kv": keys and values of ``kv_heads`` x ``head_dim`` per token in
     pages; ``window`` > 0 means only the last ``window`` positions (and the first ``keep_first``) are read, so
-    pages behind it can be given back.  kind "state": one tensor of
+    pages behind it can be given back; ``window`` < 0 that only the positions of the reader's own chunk of -window
+    positions are (chunks counted from position 0), so that the pages of finished chunks can.  kind "state": one tensor of
     ``state_shape`` per request, of fixed size, in a slot.  kind "several": the needs ``parts``
     side by side (a mixer made of several, each with a cache of its own); the mixer gets a
     ``LayerCache`` whose ``parts`` are theirs, in this order.
@@ -61,12 +62,15 @@ class CacheNeed:
 
     def widened(self, reader: "CacheNeed | None") -> "CacheNeed":
         """This need, kept for as long as ``reader`` (a layer that reads the entry without
-        writing it) also asks: the longer of the two windows, 0 standing for every key, and the more of the first keys."""
+        writing it) also asks: the longer of the two windows, 0 standing for every key, and the more of the first keys
+        (chunks of one size stay; of unequal sizes, or beside a window, every key)."""
         if reader is None or self.kind != "paged_kv":
             return self
         if (reader.kind, reader.kv_heads, reader.head_dim) != (self.kind, self.kv_heads, self.head_dim):
             raise ValueError("a layer reads a cache entry whose keys and values do not have its sizes")
         window = 0 if (self.window == 0 or reader.window == 0) else max(self.window, reader.window)
+        if min(self.window, reader.window) < 0 and self.window != reader.window:
+            window = 0
         keep = max(self.keep_first, reader.keep_first) if window else 0
         return self if (window, keep) == (self.window, self.keep_first) else CacheNeed(
             self.kind, kv_heads=self.kv_heads, head_dim=self.head_dim, window=window, keep_first=keep)
@@ -229,6 +233,18 @@ class Block(Part):
         calls the others as they are, so an arrangement that names its mixer and its
         feed-forward as steps of their own keeps the one in a graph when the other cannot be."""
         return [(bool(self.graph_safe), self.forward)]
+
+
+def joined_rows(parts: dict) -> tuple[torch.Tensor, dict]:
+    """One matrix for products of the same rows, each part from a row that is a multiple of 8 (so that kernels and products
+    can take its columns of the result where they lie; the last part is padded to a multiple of 8 too): (matrix, first row of every part)."""
+    rows, at, row = [], {}, 0
+    for name, w in parts.items():
+        at[name] = row
+        pad = -w.shape[0] % 8
+        rows += [w, torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device)]
+        row += w.shape[0] + pad
+    return torch.cat(rows, dim=0).contiguous(), at
 
 
 # ---------------------------------------------------------------------------

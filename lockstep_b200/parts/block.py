@@ -10,6 +10,8 @@ h += norm_c(mixer(norm_a(h))); h += norm_d(feed_forward(norm_b(h))).  The norms 
 ``LayerSpec.extra`` parts "mixer_post_norm" and "feed_forward_post_norm" (norms with ``accumulate``); a sublayer
 stores its result in a float32 buffer and the norm's kernel adds the normed rows to the stream, or, where the
 mixer closes with a kernel of its own that can take the norm along (``Mixer.accepts_post_norm``), that kernel does.
+Where layer norms follow one another (the one after a sublayer, then the one in front of the next sublayer, of this
+layer or of the layer that runs next), one kernel makes both: the rows wait with the step until the next sublayer takes them.
 
 "shared_norm": one norm feeds the mixer and the feed-forward side by side,
 h += mixer(y) + feed_forward(y) with y = norm(h).  Two options, each with tensors of the layer:
@@ -27,7 +29,7 @@ import torch
 from .. import kernels as K
 from ..config.spec import own_tensors, tensor_name
 from .base import Block, CacheNeed, Runtime, WeightSpec, build_part, register_part, side_stream
-from .norm import RMSNorm
+from .norm import LayerNorm, RMSNorm
 
 _DEFAULT_NAMES = {
     "mixer_norm": "input_layernorm",
@@ -122,6 +124,8 @@ class SandwichNormBlock(PreNormBlock):
         self.feed_forward_post_norm = None
         if self.feed_forward is not None:
             self.feed_forward_post_norm = build_part("norm", layer_spec.extra["feed_forward_post_norm"], runtime)
+        # the norm in front of the mixer of the layer that runs next, where the model knows which one that is
+        self.next_norm = None
         for post in (self.mixer_post_norm, self.feed_forward_post_norm):
             if post is not None and not hasattr(post, "accumulate"):
                 raise ValueError("sandwich_norm: the norm after a sublayer must be able to add its result to the stream")
@@ -130,7 +134,18 @@ class SandwichNormBlock(PreNormBlock):
         keys = list(_DEFAULT_NAMES) + ["mixer_post_norm", "feed_forward_post_norm"]
         return [(self.names[k], getattr(self, k)) for k in keys if getattr(self, k) is not None]
 
-    def _sublayer(self, part, post, x, h, ctx, cache=None):
+    def follow_with(self, block: Block) -> None:
+        """``block`` runs right after this layer, on the same stream, whenever this layer runs."""
+        # (rows cross from one layer to the next only where both are recorded together)
+        if isinstance(block, SandwichNormBlock) and self.graph_safe and block.graph_safe:
+            self.next_norm = block.mixer_norm
+
+    def _taken(self, norm, consumer, h, ctx):
+        """The rows of ``norm(h)``: made by the kernel that closed the sublayer before, or made here."""
+        rows, ctx._rows_ahead = getattr(ctx, "_rows_ahead", None), None
+        return rows if rows is not None else self._normed(norm, consumer, h)
+
+    def _sublayer(self, part, post, following, x, h, ctx, cache=None):
         args = (x, ctx, cache) if cache is not None else (x, ctx)
         if getattr(part, "accepts_post_norm", False):
             part.forward(*args, h, post_norm=post)
@@ -141,14 +156,21 @@ class SandwichNormBlock(PreNormBlock):
         else:
             K.row_bias(out, None)
             part.forward(*args, out)
-        post.accumulate(h, out)
+        if isinstance(post, LayerNorm) and isinstance(following, LayerNorm):
+            ctx._rows_ahead = post.accumulate(h, out, following)
+        else:
+            post.accumulate(h, out)
 
     def _mix(self, h, ctx, cache):
-        self._sublayer(self.mixer, self.mixer_post_norm, self._normed(self.mixer_norm, self.mixer, h), h, ctx, cache)
+        following = self.next_norm
+        if self.feed_forward is not None:
+            following = self.feed_forward_norm if self.graph_safe else None
+        self._sublayer(self.mixer, self.mixer_post_norm, following, self._taken(self.mixer_norm, self.mixer, h, ctx), h, ctx,
+                       cache)
 
     def _feed_forward(self, h, ctx, cache):
-        self._sublayer(self.feed_forward, self.feed_forward_post_norm,
-                       self._normed(self.feed_forward_norm, self.feed_forward, h), h, ctx)
+        self._sublayer(self.feed_forward, self.feed_forward_post_norm, self.next_norm,
+                       self._taken(self.feed_forward_norm, self.feed_forward, h, ctx), h, ctx)
 
 
 @register_part("block", "sandwich_norm")

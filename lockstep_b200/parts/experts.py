@@ -3,7 +3,9 @@
 Router logits z = W_router x in float32; scores from ``score`` of z ("sigmoid", or "softmax" over all
 experts, or "softmax_chosen": the logits themselves, and the weights the softmax over the chosen logits alone); the ``top`` largest scores chosen (ties to the lower index), with ``correction`` after
 adding a stored number per expert that only the choice sees; the weight of a chosen expert is its
-score (not renormalised).  ``scale`` "input": the weight multiplies what goes into the expert;
+score, or with ``renormalize`` (a number) its share of the chosen scores' sum (+ 1e-20) times that number.  ``groups`` =
+{"count", "keep"}: the experts form ``count`` equal groups of neighbours and only those of the ``keep`` best groups can be
+chosen, a group's score the sum of its two largest choice scores.  ``scale`` "input": the weight multiplies what goes into the expert;
 "output": what comes out of it.  An expert is down(act(up(.))) without biases, with ``activation``
 "relu2" (the square of relu) or "clamped_glu" (gate and up maps, g = min(gate, limit), u =
 clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1)) or "swiglu" (silu(gate) up, no clamps).  The last ``identity`` of the router's
@@ -36,7 +38,8 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, hidden_size: int, expert_size: int, experts: int, top: int, runtime: Runtime,
                  score: str = "sigmoid", activation: str = "relu2", scale: str = "input", limit: float = 0.0,
-                 alpha: float = 1.702, identity: int = 0, correction: bool = False, shared=None, names=None):
+                 alpha: float = 1.702, identity: int = 0, correction: bool = False, shared=None, names=None,
+                 renormalize: float | None = None, groups=None):
         if score not in ("sigmoid", "softmax", "softmax_chosen") or activation not in ("relu2", "clamped_glu", "swiglu") \
                 or scale not in ("input", "output"):
             raise ValueError(f"routed_experts: score {score!r}, activation {activation!r} or scale {scale!r} is not known")
@@ -45,6 +48,14 @@ class RoutedExperts(FeedForward):
         self.h, self.f, self.E, self.top, self.rt = int(hidden_size), int(expert_size), int(experts), int(top), runtime
         self.score, self.activation, self.scale = score, activation, scale
         self.limit, self.alpha, self.identity, self.correction = float(limit), float(alpha), int(identity), bool(correction)
+        if renormalize is not None and (not float(renormalize) > 0 or score == "softmax_chosen"):
+            raise ValueError("routed_experts: renormalize is a factor above zero, for scores that are not a softmax over the chosen")
+        self.pick = {"factor": float(renormalize or 0.0)}
+        if groups:
+            count, keep = int(groups["count"]), int(groups["keep"])
+            if count < 1 or (experts + identity) % count or not 1 <= keep <= count or keep * ((experts + identity) // count) < top:
+                raise ValueError(f"routed_experts: {count} groups of which {keep} are kept do not suit {top} of {experts + identity} experts")
+            self.pick.update(groups=count, keep=keep)
         self.glu = activation in ("clamped_glu", "swiglu")
         # "swiglu" is the gated unit without clamps, with the sigmoid's slope 1 and nothing added to u
         self.up_offset = 1.0
@@ -148,10 +159,10 @@ class RoutedExperts(FeedForward):
         if tokens <= K.FEW_TOKENS:
             # few tokens: the choice and the plan in one launch of one block
             K.experts_route_plan(logits, self.top, ids, weights, routed, self.score_mode, self.bias, self.E, tile,
-                                 plan, max_tiles, row_token, row_weight, pair_row, rt.err)
+                                 plan, max_tiles, row_token, row_weight, pair_row, rt.err, **self.pick)
         else:
             K.experts_route(logits, self.top, ids, weights, experts=routed, softmax=self.score_mode,
-                            correction=self.bias)
+                            correction=self.bias, **self.pick)
             K.experts_plan(ids, weights, self.E, tile, plan, max_tiles, row_token, row_weight, pair_row, rt.err)
         on_input = self.scale == "input"
         # one expert a token and nothing beside it: the second product adds into the residual stream itself (an
@@ -197,4 +208,5 @@ def _build(spec, runtime, **_):
                          score=spec.get("score", "sigmoid"), activation=spec.get("activation", "relu2"),
                          scale=spec.get("scale", "input"), limit=spec.get("limit", 0.0), alpha=spec.get("alpha", 1.702),
                          identity=spec.get("identity", 0), correction=spec.get("correction", False),
-                         shared=spec.get("shared"), names=spec.get("names"))
+                         shared=spec.get("shared"), names=spec.get("names"), renormalize=spec.get("renormalize"),
+                         groups=spec.get("groups"))

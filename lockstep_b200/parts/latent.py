@@ -11,11 +11,13 @@ Since q_plain,h . (W_uk,h c) = (W_uk,h^T q_plain,h) . c, the attention kernels a
 [c ; k_rot] (padded to a multiple of 16) that every query head reads, queries
 [W_uk,h^T q_plain,h ; q_rot,h], and values [c ; 0]; the head's output, a weighted sum of latents, then
 goes through W_uv,h.  A prompt's tokens and a decoded token take the same path, so a row does not
-depend on how its request was cut.  Rotation is the position encoding's (its tables; neighbouring
+depend on how its request was cut.  Without ``rot_dim`` nothing is rotated.  Rotation is the position encoding's (its tables; neighbouring
 pairs or halves), a window and a sink per head are optional.
 
 ``q_rank``: the queries go through a latent of their own, q = W_uq norm(W_dq x) with an RMSNorm (a gain
 per element) between the two maps (``names``: ``q_down``, ``q_norm``, ``q_up``), instead of one matrix ``q``.
+``gate``: the heads' outputs are multiplied, element by element, by sigmoid(W_g x) (``names``: ``gate``) before the output
+projection; W_g's rows ride on the first product, the multiplication on the product with W_uv.
 ``borrows_kv``: the layer has no down-projection of its own; the schedule gives it the cached latents and
 rotated key parts of another layer, which it reads with its own W_uk, W_uv, queries and scale.
 
@@ -30,11 +32,11 @@ import torch
 
 from .. import kernels as K
 from .attention import ScoreExtras, attend
-from .base import CacheNeed, Mixer, PositionEncoding, Runtime, WeightSpec, register_part
+from .base import CacheNeed, Mixer, PositionEncoding, Runtime, WeightSpec, joined_rows, register_part
 from .norm import NormedRows
 
 _DEFAULT_NAMES = {"q": "q", "down": "dkv", "down_norm": "dkv.norm", "up_k": "uk", "up_v": "uv", "o": "o",
-                  "sink": "sink", "q_down": "dq", "q_norm": "dq.norm", "q_up": "uq"}
+                  "sink": "sink", "gate": "g", "q_down": "dq", "q_norm": "dq.norm", "q_up": "uq"}
 
 
 class LatentAttention(Mixer):
@@ -43,10 +45,11 @@ class LatentAttention(Mixer):
     can_overwrite = True
 
     def __init__(self, hidden_size, num_heads, head_dim, rot_dim, value_dim, kv_rank, scale, window, norm_eps,
-                 position: PositionEncoding, runtime: Runtime, sink=False, names=None, q_rank=None, borrows_kv=False):
+                 position: PositionEncoding, runtime: Runtime, sink=False, names=None, q_rank=None, borrows_kv=False,
+                 gate=False):
         self.w, self.H, self.d, self.dr = int(hidden_size), int(num_heads), int(head_dim), int(rot_dim)
         self.dv, self.rank = int(value_dim), int(kv_rank)
-        self.q_rank, self.borrows = int(q_rank or 0), bool(borrows_kv)
+        self.q_rank, self.borrows, self.gated = int(q_rank or 0), bool(borrows_kv), bool(gate)
         self.scale, self.window, self.eps = float(scale), int(window or 0), float(norm_eps)
         self.sink, self.position, self.rt = bool(sink), position, runtime
         self.pad = -(-(self.rank + self.dr) // 16) * 16          # the one head size the attention kernels see
@@ -80,6 +83,8 @@ class LatentAttention(Mixer):
         if not self.borrows:
             specs.update({n["down"]: WeightSpec((self.rank + self.dr, self.w)),
                           n["down_norm"]: WeightSpec((self.rank,), "gain")})
+        if self.gated:
+            specs[n["gate"]] = WeightSpec((H * self.dv, self.w))
         if self.sink:
             specs[n["sink"]] = WeightSpec((H,), "gain", ("normal", 0.0, 1.0))
         return specs
@@ -87,15 +92,18 @@ class LatentAttention(Mixer):
     def bind(self, t):
         n, H = self.names, self.H
         # one product for what reads the mixer's input: the queries and, where the layer makes them itself, the
-        # latent and the shared key part.  Queries through a latent of their own: that latent is a product of
+        # latent and the shared key part, and the output gate's logits.  Queries through a latent of their own: that latent is a product of
         # its own with a float32 result, which its norm reads as it is.
-        self.w_in = None
+        parts = []
         if self.q_rank:
             self.w_q_down, self.q_gain, self.w_q_up = t[n["q_down"]].contiguous(), t[n["q_norm"]], t[n["q_up"]].contiguous()
-            if not self.borrows:
-                self.w_in = t[n["down"]].contiguous()
         else:
-            self.w_in = t[n["q"]].contiguous() if self.borrows else torch.cat([t[n["q"]], t[n["down"]]], dim=0).contiguous()
+            parts.append(("q", t[n["q"]]))
+        if not self.borrows:
+            parts.append(("kv", t[n["down"]]))
+        if self.gated:
+            parts.append(("gate", t[n["gate"]]))
+        self.w_in, self.at = joined_rows(dict(parts)) if parts else (None, {})
         self.gain = None if self.borrows else t[n["down_norm"]]
         # W_uk per head, transposed: [H, rank, d], so that the fold is a product with rows of weights
         self.w_fold = t[n["up_k"]].view(H, self.d, self.rank).transpose(1, 2).contiguous()
@@ -127,9 +135,9 @@ class LatentAttention(Mixer):
                 cq = rt.rows(t, self.q_rank)
                 K.rmsnorm(raw, self.q_gain, cq, self.eps, rt.err)
                 K.gemm_nt(cq, self.w_q_up, queries, err=rt.err)
-            kv = proj
         else:
-            queries, kv = proj, None if self.borrows else proj[:, H * (self.d + self.dr):]
+            queries = proj
+        kv = None if self.borrows else proj[:, self.at["kv"]:self.at["kv"] + self.rank + self.dr]
         rot = self.position.rotary() if self.dr else None
         cos, sin, _ = rot if rot is not None else (None, None, 0)
         q = rt.rows(t, H * self.pad)
@@ -143,7 +151,8 @@ class LatentAttention(Mixer):
             K.heads_product(queries, self.d + self.dr, self.w_fold, q, self.pad)
         attn = attend(rt, q, ctx, cache, H, 1, self.pad, self.window, self.scale, self.exact, self.extras)
         y = rt.rows(t, H * self.dv)
-        K.heads_product(attn, self.pad, self.w_up_v, y, self.dv)
+        gate = proj[:, self.at["gate"]:self.at["gate"] + H * self.dv] if self.gated else None
+        K.heads_product(attn, self.pad, self.w_up_v, y, self.dv, gate=gate)
         K.gemm_nt(y, self.w_o, residual, K.EPILOGUE_STORE if overwrite else K.EPILOGUE_RESIDUAL, err=rt.err)
 
 
@@ -152,4 +161,5 @@ def _build(spec, runtime, position=None, **_):
     return LatentAttention(spec["hidden_size"], spec["num_heads"], spec["head_dim"], spec["rot_dim"],
                            spec["value_dim"], spec["kv_rank"], spec["scale"], spec.get("window", 0), spec["norm_eps"],
                            position, runtime, sink=spec.get("sink", False), names=spec.get("names"),
-                           q_rank=spec.get("q_rank"), borrows_kv=spec.get("borrows_kv", False))
+                           q_rank=spec.get("q_rank"), borrows_kv=spec.get("borrows_kv", False),
+                           gate=spec.get("gate", False))

@@ -127,14 +127,19 @@ class GatedUnit(FeedForward):
 
 
 class PlainUnit(FeedForward):
-    """down(gelu_tanh(up(x))) without biases and without a gate; the activation is made in the first product's epilogue."""
+    """down(act(up(x))) without biases and without a gate, ``activation`` "gelu_tanh" or "relu2" (the square of relu),
+    made in the first product's epilogue."""
 
     graph_safe = True
     accepts_normed_rows = True
     can_overwrite = True
 
-    def __init__(self, hidden_size: int, intermediate_size: int, runtime: Runtime, names=None):
-        self.h, self.i, self.rt = int(hidden_size), int(intermediate_size), runtime
+    EPILOGUES = {"gelu_tanh": K.EPILOGUE_GELU, "relu2": K.EPILOGUE_RELU2}
+
+    def __init__(self, hidden_size: int, intermediate_size: int, runtime: Runtime, names=None, activation: str = "gelu_tanh"):
+        if activation not in self.EPILOGUES:
+            raise ValueError(f"plain_unit: activation {activation!r} is not known ({', '.join(self.EPILOGUES)})")
+        self.h, self.i, self.rt, self.epilogue = int(hidden_size), int(intermediate_size), runtime, self.EPILOGUES[activation]
         self.names = {"up": "up", "down": "down"}
         self.names.update(names or {})
         self.w_up = self.w_down = None
@@ -148,15 +153,16 @@ class PlainUnit(FeedForward):
     def forward(self, x, ctx, residual, overwrite=False):
         act = self.rt.rows(residual.shape[0], self.i)
         if isinstance(x, NormedRows):
-            x.linear(self.w_up, act, K.EPILOGUE_GELU, self.rt.err)
+            x.linear(self.w_up, act, self.epilogue, self.rt.err)
         else:
-            K.gemm_nt(x, self.w_up, act, K.EPILOGUE_GELU, err=self.rt.err)
+            K.gemm_nt(x, self.w_up, act, self.epilogue, err=self.rt.err)
         K.gemm_nt(act, self.w_down, residual, K.EPILOGUE_STORE if overwrite else K.EPILOGUE_RESIDUAL, err=self.rt.err)
 
 
 @register_part("feed_forward", "plain_unit")
 def _build_plain_unit(spec, runtime, **_):
-    return PlainUnit(spec["hidden_size"], spec["intermediate_size"], runtime, names=spec.get("names"))
+    return PlainUnit(spec["hidden_size"], spec["intermediate_size"], runtime, names=spec.get("names"),
+                     activation=spec.get("activation", "gelu_tanh"))
 
 
 @register_part("feed_forward", "gated_unit")

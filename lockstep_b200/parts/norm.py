@@ -6,9 +6,10 @@ own prefix names it).  ``groups`` > 1: the row is cut into that many equal conse
 each is divided by its own root mean square (the gain still runs over the whole row).  ``scalar``:
 the stored gain is one number for all coordinates (a tensor without dimensions).
 
-"layernorm": y = (x - mean) * rsqrt(var + eps) * gain with var the mean of the squared deviations and no bias,
-all in float32.  ``accumulate(residual, x)`` adds the norm of float32 rows ``x`` to ``residual`` (a norm that
-follows a sublayer)."""
+"layernorm": y = (x - mean) * rsqrt(var + eps) * gain (+ bias) with var the mean of the squared deviations,
+all in float32.  ``bias``: the local name of the stored bias (absent: none).  ``accumulate(residual, x)`` adds the norm of
+float32 rows ``x`` to ``residual`` (a norm that follows a sublayer); with ``follow``, a layer norm that the next sublayer
+begins with, the same kernel norms the new stream with it and the rows are returned."""
 
 from __future__ import annotations
 
@@ -88,27 +89,37 @@ def _build(spec, runtime, **_):
 class LayerNorm(Norm):
     graph_safe = True
 
-    def __init__(self, width: int, eps: float, runtime: Runtime, tensor: str = "weight"):
-        self.width, self.eps, self.rt, self.tensor = int(width), float(eps), runtime, str(tensor)
+    def __init__(self, width: int, eps: float, runtime: Runtime, tensor: str = "weight", bias: str | None = None):
+        self.width, self.eps, self.rt, self.tensor, self.bias_tensor = int(width), float(eps), runtime, str(tensor), bias
         self.gain: torch.Tensor | None = None
+        self.bias: torch.Tensor | None = None
 
     def weight_specs(self):
-        return {self.tensor: WeightSpec((self.width,), "gain")}
+        specs = {self.tensor: WeightSpec((self.width,), "gain")}
+        if self.bias_tensor is not None:
+            specs[self.bias_tensor] = WeightSpec((self.width,), "gain", ("normal", 0.0, 0.02))
+        return specs
 
     def bind(self, tensors):
         self.gain = tensors[self.tensor].to(torch.float32).contiguous()
+        if self.bias_tensor is not None:
+            self.bias = tensors[self.bias_tensor].to(torch.float32).contiguous()
 
     def forward(self, h, row_index=None):
         rows = h.shape[0] if row_index is None else row_index.numel()
         out = self.rt.rows(rows, self.width)
-        K.layernorm(h, self.gain, out, self.eps, self.rt.err, row_index)
+        K.layernorm(h, self.gain, out, self.eps, self.rt.err, row_index, bias=self.bias)
         return out
 
-    def accumulate(self, residual, x):
-        """residual += norm(x); both float32 [rows, width]."""
-        K.norm_merge_add(residual, x.view(1, *x.shape), None, 1.0, self.gain, 0.0, self.eps)
+    def accumulate(self, residual, x, follow: "LayerNorm | None" = None):
+        """residual += norm(x); both float32 [rows, width].  With ``follow``: the rows of follow(residual), of the
+        engine's type, made in the same kernel."""
+        out = self.rt.rows(residual.shape[0], self.width) if follow is not None else None
+        K.norm_merge_add(residual, x.view(1, *x.shape), None, 1.0, self.gain, 0.0, self.eps, post_bias=self.bias,
+                         follow=(follow.gain, follow.bias, follow.eps, out) if follow is not None else None)
+        return out
 
 
 @register_part("norm", "layernorm")
 def _build_layernorm(spec, runtime, **_):
-    return LayerNorm(spec["width"], spec["eps"], runtime, spec.get("tensor", "weight"))
+    return LayerNorm(spec["width"], spec["eps"], runtime, spec.get("tensor", "weight"), spec.get("bias"))

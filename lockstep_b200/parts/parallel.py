@@ -91,7 +91,8 @@ class ParallelMixers(Mixer):
             K.weighted_sum(residual, out, self.scales, self.bias if self.overwrite else None)
             return
         post = (post_norm.gain, post_norm.eps) if post_norm is not None else (None, 0.0)
-        K.norm_merge_add(residual, out, self.branch_gain, self.scales[0], post[0], float(self.branch_norm["eps"]), post[1])
+        K.norm_merge_add(residual, out, self.branch_gain, self.scales[0], post[0], float(self.branch_norm["eps"]), post[1],
+                         post_bias=post_norm.bias if post_norm is not None else None)
 
     def forward(self, x, ctx, cache, residual, post_norm=None):
         n, t = len(self.mixers), residual.shape[0]

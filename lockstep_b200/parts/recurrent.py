@@ -52,7 +52,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels as K
-from .base import CacheNeed, Mixer, Runtime, WeightSpec, register_part
+from .base import CacheNeed, Mixer, Runtime, WeightSpec, joined_rows, register_part
 from .norm import NormedRows
 
 
@@ -71,18 +71,6 @@ def portion_list(ctx, state: torch.Tensor, rt: Runtime):
 
 def _f32(t: torch.Tensor) -> torch.Tensor:
     return t.to(torch.float32).contiguous()
-
-
-def _joined(parts: dict) -> tuple[torch.Tensor, dict]:
-    """One matrix for products of the same rows, each part from a row that is a multiple of 8 (so that kernels and products
-    can take its columns of the result where they lie): (matrix, first row of every part)."""
-    rows, at, row = [], {}, 0
-    for name, w in parts.items():
-        at[name] = row
-        pad = -w.shape[0] % 8
-        rows += [w, torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device)]
-        row += w.shape[0] + pad
-    return torch.cat(rows, dim=0).contiguous(), at
 
 
 def _product(x, w, out, err) -> None:
@@ -146,7 +134,7 @@ class GatedDelta(Mixer):
         self.w_o, self.dt_bias, self.a_log, self.gain = t["o"], _f32(t["dt_bias"]), _f32(t["A_log"]), _f32(t["norm"])
         if self.per_head:
             # one product for q, k, v and the gate, and one with a float32 result for beta's and the decay's logits
-            self.w_in, self.at = _joined({"qkv": torch.cat([t["q"], t["k"], t["v"]], dim=0), "g": t["g"]})
+            self.w_in, self.at = joined_rows({"qkv": torch.cat([t["q"], t["k"], t["v"]], dim=0), "g": t["g"]})
             self.w_gates = torch.cat([t["b"], t["a"]], dim=0).contiguous()
             return
         if t["a1"].shape[0] != t["a2"].shape[1] or t["g1"].shape[0] != t["g2"].shape[1]:
@@ -482,7 +470,7 @@ class MLstm(Mixer):
 
     def bind(self, t):
         n = self.names
-        self.w_in, self.at = _joined({s: t[n[s]] for s in ("q", "k", "v", "g")})
+        self.w_in, self.at = joined_rows({s: t[n[s]] for s in ("q", "k", "v", "g")})
         # the gates' logits are a product of their own, with a float32 result
         self.w_gates = torch.cat([t[n["i"]], t[n["f"]]], dim=0).contiguous()
         self.gate_bias = _f32(torch.cat([t[n["i_bias"]], t[n["f_bias"]]]))

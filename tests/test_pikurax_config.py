@@ -55,7 +55,7 @@ def test_cache_needs_in_the_manager():
     needs = model.cache_needs()
     assert len(needs) == 9 and model.embedding_entry == 8               # eight runs and the embedding's last token
     assert needs[8].kind == "state" and needs[8].state_dtype == torch.int32
-    assert needs[0].kind == "several" and needs[0].parts[0].window == 0  # a chunked layer keeps every page
+    assert needs[0].kind == "several" and needs[0].parts[0].window == -24  # a chunked layer keeps the pages of the running chunk
     assert needs[0].parts[1].state_shape == (4 * 40,)                    # S and three carried inputs
     assert needs[1].parts[0].head_dim == 32 and needs[1].parts[1].state_shape == (3 * 8 * 24,)
     cm = CacheManager(needs, num_pages=8, page_size=16, max_live=2, max_seq_len=64, allocate=False)
