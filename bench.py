@@ -39,6 +39,8 @@ two of the layers run twice) beside Qwen3 layers of equal width, depth, head cou
 feed-forward size.
 ``--workload pikurax`` does the same for the Pikurax design beside Malazen.
 ``--workload kusolorn`` does the same for the Kusolorn design beside Sevipel and Malazen.
+``--workload tesozen`` does the same for the Tesozen design (differential attention, a matrix memory, attention over a
+cached latent with a gate, layer norms around every sublayer, group-limited experts) beside Kusolorn, Kemirax and Pikurax.
 ``--workload kemirax`` does the same for the Kemirax design (one norm feeding a mixer behind a token
 shift and routed experts side by side, gates on both; attention over a cached latent with queries
 through a latent and layers that read another layer's cache; gated linear attention; identity and
@@ -578,7 +580,7 @@ def kernel_times(runner, entries_of, steps=3):
              "experts_product_tc", "experts_gather", "experts_combine", "latent_finish", "heads_product",
              "sigmoid_power_decay", "clamped_glu", "row_bias", "weighted_sum", "gated_sum", "experts_mix", "rmsnorm_shift", "experts_route_plan",
              "layernorm", "norm_merge_add", "pair_embed", "rows_cast", "scale_cap", "unit_gates", "unit_scan", "rotate_rows",
-             "side_gate", "side_gate_few"]
+             "side_gate", "side_gate_few", "map_difference", "map_difference_fold"]
     records, saved, graphs, turn = [], {}, runner.graphs, [0]
     runner.graphs = None
 
@@ -1222,6 +1224,134 @@ def run_kusolorn(args):
     return 0
 
 
+TESOZEN_SIZES = {
+    "w1024": {"width": 1024, "heads": 8, "kv_heads": 4, "linear_heads": 4, "latent_heads": 8, "experts": 32, "groups": 8, "keep": 4,
+              "top": 4, "expert_ff": 512, "shared_ff": 1024, "ff": 4096},
+    "w2048": {"width": 2048, "heads": 16, "kv_heads": 4, "linear_heads": 8, "latent_heads": 16, "experts": 32, "groups": 8, "keep": 4,
+              "top": 4, "expert_ff": 1024, "shared_ff": 2048, "ff": 8192},
+}
+TESOZEN_RANK, TESOZEN_CHUNK = 128, 1024
+
+
+def tesozen_config(z):
+    """Eight layers: three with differential attention (values of 128 elements and two maps of 64, so that a head's cache row is
+    that of a head of 128; Pikurax's chunks of this file), three with Kusolorn's matrix memory, two over a latent of as many
+    elements as Kemirax's latent and rotated part together; half have Kusolorn's dense feed-forward, half experts of Kemirax's
+    sizes with its shared expert."""
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "shared": {"ff": z["shared_ff"]},
+           "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": z["groups"], "keep": z["keep"]}, "scale": 2.5}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.4,
+           "mask": {"size": TESOZEN_CHUNK}}
+    lstm = {"heads": z["linear_heads"], "dim": 128, "vdim": 128, "gate_cap": 15.0}
+    lat = {"heads": z["latent_heads"], "dim": MALAZEN_PLAIN, "vdim": MALAZEN_VALUE, "kv_rank": TESOZEN_RANK,
+           "scale": MALAZEN_PLAIN ** -0.5}
+    kinds = [("attention", att, dense), ("mlstm", lstm, moe), ("latent_attention", lat, dense), ("attention", att, moe),
+             ("mlstm", lstm, dense), ("latent_attention", lat, moe), ("attention", att, dense), ("mlstm", lstm, moe)]
+    return {"architecture": "Tesozen", "vocab": DESIGN_VOCAB, "width": z["width"], "norm": {"eps": 1e-5}, "max_positions": 4096,
+            "embedding": {"scale": 8.0},
+            "layers": [{"type": t, "mixer": json.loads(json.dumps(m)), "mlp": json.loads(json.dumps(f))} for t, m, f in kinds]}
+
+
+def run_tesozen(args):
+    pk = peaks()
+    tokens, batch, context = PREFILL_TOKENS, 8, DESIGN_CONTEXT
+    sizes = {}
+    clocks = ClockSampler()
+    clocks.start()
+    for size, z in TESOZEN_SIZES.items():
+        kz, ez, pz = KUSOLORN_SIZES[size], KEMIRAX_SIZES[size], PIKURAX_SIZES[size]
+        row = {"tesozen": measure_design(tesozen_config(z), args, tokens, batch, context),
+               "kusolorn": measure_design(kusolorn_config(kz), args, tokens, batch, context),
+               "kemirax": measure_design(kemirax_config(ez), args, tokens, batch, context),
+               "pikurax": measure_design(pikurax_config(pz), args, tokens, batch, context)}
+        w, H, G, LH, QH, ff = z["width"], z["heads"], z["kv_heads"], z["linear_heads"], z["latent_heads"], z["ff"]
+        R, DP, DV, F, SF = TESOZEN_RANK, MALAZEN_PLAIN, MALAZEN_VALUE, z["expert_ff"], z["shared_ff"]
+        n_att, n_lstm, n_lat, n_dense, n_moe = 3, 3, 2, 4, 4
+        # products of a prefill through the engine's product kernels (experts and per-head products apart)
+        lstm_cols = 5 * LH * 128 + 2 * LH
+        flops_t = 2 * tokens * w * (n_att * ((2 * H + 2 * G) * 128 + H) + n_lstm * lstm_cols + n_lat * (QH * (DP + 2 * DV) + R)
+                                    + n_dense * 2 * ff + n_moe * (z["experts"] + 3 * SF)) + 2 * DESIGN_VOCAB * w
+        k_cols = 3 * lstm_cols + 3 * (2 * kz["kv_heads"] * 128 + 3 * kz["heads"] * 128 + 2 * kz["heads"]) \
+            + 2 * (2 * kz["heads"] + 2 * kz["kv_heads"]) * 128 + 4 * 2 * kz["ff"] + 4 * kz["experts"] + 8 * 2 * kz["side"]
+        flops_k = 2 * tokens * w * k_cols + 2 * DESIGN_VOCAB * w
+        pairs_full = tokens * (tokens + 1) // 2
+        pairs_chunk = sum(i % TESOZEN_CHUNK + 1 for i in range(tokens))
+        pairs_win = sum(min(i + 1, kz["window"]) + min(max(i + 1 - kz["window"], 0), KUSOLORN_KEPT) for i in range(tokens))
+        # a pair of a query head and a key: two maps of 64 elements and two sums over 128
+        att_t = n_att * 2 * (2 * 64 + 2 * 128) * pairs_chunk * H + n_lat * 4 * pairs_full * QH * R
+        att_k = 2 * 4 * pairs_win * H * 128
+        att_e = 5 * 4 * pairs_full * QH * (MALAZEN_RANK + MALAZEN_ROT)
+        att_p = 4 * H * 128 * (4 * pairs_chunk + 4 * pairs_full)
+        up = lambda top, f, layers: 2 * tokens * top * 2 * f * w * layers
+        real = ez["top"] * ez["experts"] / (ez["experts"] + ez["identity"])
+        cache_t = 2 * batch * (n_att * (context % TESOZEN_CHUNK or TESOZEN_CHUNK) * 2 * G * 128 + n_lat * context * 2 * R)
+        cache_k = 2 * batch * 2 * (kz["window"] + KUSOLORN_KEPT) * 2 * G * 128
+        cache_e = 2 * batch * 5 * context * 2 * (MALAZEN_RANK + MALAZEN_ROT)
+        state = 2 * 4 * batch * 3 * LH * 128 * 128
+        stream = 4 * tokens * w                     # one float32 pass over the step's rows
+
+        def frac(amount, ms, peak):
+            return round(amount / (ms * 1e-3) / peak, 4) if ms else None
+
+        def ms_of(kernels, *names):
+            return sum(kernels.get(n, 0.0) for n in names)
+
+        tf, bw = pk["bf16_tflops"] * 1e12, pk["hbm_gbs"] * 1e9
+        products = ("gemm_nt_tc", "gemm_nt_tc_rmsnorm")
+        attention = ("attention_tile", "attention_prefill_tc")
+        decode_attention = ("attention_decode", "attention_decode_mma", "attention_tile")
+        tp, kp, ep, pp = (row[d]["prefill_kernels_ms"] for d in ("tesozen", "kusolorn", "kemirax", "pikurax"))
+        td, kd, ed, pd = (row[d]["decode_kernels_ms"] for d in ("tesozen", "kusolorn", "kemirax", "pikurax"))
+        per_token = lambda kernels, name, layers: round(ms_of(kernels, name) * 1e3 / (layers * tokens), 4)
+        row["like_kernels_fraction_of_measured_peak [tesozen, like kernel]"] = {
+            "prefill: products (tensor cores); kusolorn": [frac(flops_t, ms_of(tp, *products), tf), frac(flops_k, ms_of(kp, *products), tf)],
+            "prefill: attention; kusolorn, kemirax, pikurax": [frac(att_t, ms_of(tp, *attention), tf), frac(att_k, ms_of(kp, *attention), tf),
+                                                               frac(att_e, ms_of(ep, *attention), tf), frac(att_p, ms_of(pp, *attention), tf)],
+            "prefill: mlstm rule, microseconds a token and layer; kusolorn": [per_token(tp, "mlstm_rule", 3), per_token(kp, "mlstm_rule", 3)],
+            "prefill: per-head products of the latent (of the bf16 peak); kemirax": [
+                frac(n_lat * 2 * tokens * QH * R * (DP + DV), ms_of(tp, "heads_product"), tf),
+                frac(5 * 2 * tokens * QH * MALAZEN_RANK * (DP + DV), ms_of(ep, "heads_product"), tf)],
+            "prefill: experts' first product; kemirax": [frac(up(z["top"], F, n_moe), ms_of(tp, "experts_up"), tf),
+                                                         frac(up(real, F, 8), ms_of(ep, "experts_up"), tf)],
+            "prefill: experts' second product; kemirax": [frac(up(z["top"], F, n_moe) / 2, ms_of(tp, "experts_down"), tf),
+                                                          frac(up(real, F, 8) / 2, ms_of(ep, "experts_down"), tf)],
+            "prefill: gated activations (bytes read and written); kemirax": [
+                frac(n_moe * tokens * (z["top"] * F + SF) * 10, ms_of(tp, "clamped_glu"), bw),
+                frac(8 * tokens * (real * F + SF) * 10, ms_of(ep, "clamped_glu"), bw)],
+            "prefill: choice, microseconds a launch (groups); kemirax": [round(ms_of(tp, "experts_route") * 1e3 / n_moe, 2),
+                                                                          round(ms_of(ep, "experts_route") * 1e3 / 8, 2)],
+            "prefill: experts' sum (bytes); kemirax": [
+                frac(n_moe * stream * (z["top"] + 2), ms_of(tp, "experts_mix"), bw),
+                frac(8 * stream * (real + 2), ms_of(ep, "experts_mix"), bw)],
+            "prefill: q, k, v finished (qkv_finish; bytes read and written); kusolorn": [
+                frac(n_att * tokens * ((H + 2 * G) * 128 * 2 + (2 * H + 2 * G) * 128 * 2), ms_of(tp, "qkv_finish"), bw),
+                frac(2 * tokens * (H + 2 * G) * 128 * 4, ms_of(kp, "qkv_finish"), bw)],
+            "prefill: difference of two maps (map_difference; bytes); kusolorn's head_rms_gate": [
+                frac(n_att * tokens * H * 128 * 6, ms_of(tp, "map_difference"), bw),
+                frac(tokens * 8 * 128 * 3 * (LH + H), ms_of(kp, "head_rms_gate"), bw)],
+            "prefill: read-out's norm and gate (head_rms_gate); kusolorn": [
+                frac(tokens * 8 * 128 * 3 * LH, ms_of(tp, "head_rms_gate"), bw),
+                frac(tokens * 8 * 128 * 3 * (LH + H), ms_of(kp, "head_rms_gate"), bw)],
+            "prefill: a sublayer's closing kernel (3 passes, with the next norm 3.5); pikurax (4 or 3), whose norms are kernels of their own": [
+                frac(16 * 3.5 * stream, ms_of(tp, "norm_merge_add"), bw), frac((8 * 4 + 8 * 3) * stream, ms_of(pp, "norm_merge_add"), bw)],
+            "decode: attention (bytes of cache); kusolorn, kemirax": [
+                frac(cache_t, ms_of(td, *decode_attention), bw), frac(cache_k, ms_of(kd, *decode_attention), bw),
+                frac(cache_e, ms_of(ed, *decode_attention), bw)],
+            "decode: mlstm rule (bytes of state); kusolorn": [frac(state, ms_of(td, "mlstm_rule"), bw), frac(state, ms_of(kd, "mlstm_rule"), bw)],
+            "decode: milliseconds of [map_difference_fold; kusolorn's attention_combine]": [
+                round(ms_of(td, "map_difference_fold"), 4), round(ms_of(kd, "attention_combine"), 4)],
+        }
+        sizes[size] = row
+    clock = clocks.stop()
+    print(json.dumps({
+        "metric": "prefill of 2,048 tokens and decode at batch 8, context 2,048: Tesozen beside Kusolorn, Kemirax and Pikurax at equal size",
+        "unit": "ms, tok/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic", "impl": "ours", "clocks": clock,
+        "peaks": pk, "layer_runs": 8, "vocab": DESIGN_VOCAB, "sizes": sizes,
+    }))
+    return 0
+
+
 # ---------------------------------------------------------------------------
 # the reference arm: LockStep itself, unmodified, from baseline/_ref
 # ---------------------------------------------------------------------------
@@ -1391,9 +1521,9 @@ def main():
     ap.add_argument("--no-fp32", action="store_true", help="skip the float32 points")
     ap.add_argument("--only", default="", choices=["", "decode", "prefill"],
                     help="time only this part and print a short line (for profiling a small case)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "designs", "malazen", "kemirax", "pikurax", "kusolorn"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "mixed", "designs", "malazen", "kemirax", "pikurax", "kusolorn", "tesozen"],
                     help="mixed: a continuous batch of 64 requests through the entry point; designs: the Sevipel "
-                         "design beside Qwen3 layers of equal size, with every kernel's time; malazen, kemirax, pikurax, kusolorn: the same "
+                         "design beside Qwen3 layers of equal size, with every kernel's time; malazen, kemirax, pikurax, kusolorn, tesozen: the same "
                          "for those designs")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
                     help="element type of the --only runs (the full line always reports both)")
@@ -1420,6 +1550,8 @@ def main():
         return run_pikurax(args)
     if args.workload == "kusolorn":
         return run_kusolorn(args)
+    if args.workload == "tesozen":
+        return run_tesozen(args)
     return run_ours(args)
 
 

@@ -12,6 +12,8 @@
 // may differ from run to run, but no value depends on it: every element of a product is one
 // chain of fused multiply-adds over ascending k, whatever tile its row lies in, and a token's
 // choices are added in order of rank.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace {
@@ -33,15 +35,16 @@ constexpr int TILE_M = 64, TILE_N = 64, TILE_K = 16;
 // pick: groups > 0: only experts of the `keep` best of that many equal groups of neighbours can be chosen, a group's
 // score the sum of its two largest choice scores (ties to the lower group); factor > 0: the weights are divided by
 // (their sum over the chosen, in order of rank, + 1e-20) and multiplied by it.
-// (one warp: token t)
+// (one warp: token t; PL: experts a lane looks after)
+template <int PL>
 __device__ __forceinline__ void route_token(const float* __restrict__ logits, int64_t ld, int t, int experts, int top,
                                             int softmax, const float* __restrict__ correction, const RoutePick rule,
                                             int* __restrict__ ids, float* __restrict__ weights) {
   const int lane = threadIdx.x & 31;
-  float z[MAX_PER_LANE];     // the expert's score
-  float pick[MAX_PER_LANE];  // what the choice compares
+  float z[PL];     // the expert's score
+  float pick[PL];  // what the choice compares
 #pragma unroll
-  for (int i = 0; i < MAX_PER_LANE; ++i) {
+  for (int i = 0; i < PL; ++i) {
     const int e = lane + 32 * i;
     z[i] = e < experts ? logits[(int64_t)t * ld + e] : -INFINITY;
   }
@@ -50,37 +53,37 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
   } else if (softmax) {
     float top_z = -INFINITY;
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) top_z = fmaxf(top_z, z[i]);
+    for (int i = 0; i < PL; ++i) top_z = fmaxf(top_z, z[i]);
     top_z = ls_warp_max(top_z);
     float sum = 0.f;
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) {
+    for (int i = 0; i < PL; ++i) {
       z[i] = lane + 32 * i < experts ? expf(z[i] - top_z) : 0.f;
       sum += z[i];
     }
     sum = ls_warp_sum(sum);
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) z[i] = z[i] / sum;
+    for (int i = 0; i < PL; ++i) z[i] = z[i] / sum;
   } else {
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) z[i] = 1.0f / (1.0f + expf(-z[i]));
+    for (int i = 0; i < PL; ++i) z[i] = 1.0f / (1.0f + expf(-z[i]));
   }
 #pragma unroll
-  for (int i = 0; i < MAX_PER_LANE; ++i) {
+  for (int i = 0; i < PL; ++i) {
     const int e = lane + 32 * i;
     pick[i] = e < experts ? (correction != nullptr ? z[i] + correction[e] : z[i]) : -INFINITY;
   }
   if (rule.groups > 0) {
     // lane g % 32 keeps the score of group g in place g / 32; the choice then takes the best groups one by one
     const int size = experts / rule.groups;
-    float group_score[MAX_PER_LANE];
+    float group_score[PL];
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) group_score[i] = -INFINITY;
+    for (int i = 0; i < PL; ++i) group_score[i] = -INFINITY;
     for (int g = 0; g < rule.groups; ++g) {
       const int from = g * size, to = from + size;
       float a = -INFINITY, b = -INFINITY;              // the largest and the second of this lane's experts of the group
 #pragma unroll
-      for (int i = 0; i < MAX_PER_LANE; ++i) {
+      for (int i = 0; i < PL; ++i) {
         const int e = lane + 32 * i;
         if (e >= from && e < to) {
           b = fmaxf(b, fminf(a, pick[i]));
@@ -95,7 +98,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
       }
       const float score = size > 1 ? a + b : a;
 #pragma unroll
-      for (int i = 0; i < MAX_PER_LANE; ++i)
+      for (int i = 0; i < PL; ++i)
         if (lane + 32 * i == g) group_score[i] = score;
     }
     unsigned open = 0;                                 // this lane's experts whose group is kept
@@ -103,7 +106,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
       float best = -INFINITY;
       int at = 0x7fffffff;
 #pragma unroll
-      for (int i = 0; i < MAX_PER_LANE; ++i) {
+      for (int i = 0; i < PL; ++i) {
         const int g = lane + 32 * i;
         if (g < rule.groups && (group_score[i] > best || (group_score[i] == best && g < at))) {
           best = group_score[i];
@@ -119,14 +122,14 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
         }
       }
 #pragma unroll
-      for (int i = 0; i < MAX_PER_LANE; ++i) {
+      for (int i = 0; i < PL; ++i) {
         const int e = lane + 32 * i;
         if (e == at) group_score[i] = -INFINITY;       // (as a group: taken)
         if (e >= at * size && e < (at + 1) * size) open |= 1u << i;
       }
     }
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i)
+    for (int i = 0; i < PL; ++i)
       if (!((open >> i) & 1u)) pick[i] = -INFINITY;
   }
   unsigned taken = 0;
@@ -134,7 +137,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
     float best = -INFINITY, best_z = 0.f;
     int at = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) {
+    for (int i = 0; i < PL; ++i) {
       const int e = lane + 32 * i;
       if (e < experts && !((taken >> i) & 1u) && (pick[i] > best || (pick[i] == best && e < at))) {
         best = pick[i];
@@ -177,6 +180,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, in
   }
 }
 
+template <int PL>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_kernel(const float* __restrict__ logits, int64_t ld, int tokens,
                                                                  int experts, int top, int softmax,
                                                                  const float* __restrict__ correction, RoutePick rule,
@@ -184,7 +188,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_kernel(const float* __
   ls_dependency_sync();
   const int t = blockIdx.x * ROUTE_WARPS + (threadIdx.x >> 5);
   if (t >= tokens) return;
-  route_token(logits, ld, t, experts, top, softmax, correction, rule, ids, weights);
+  route_token<PL>(logits, ld, t, experts, top, softmax, correction, rule, ids, weights);
 }
 
 // plan [0] = tiles, then (expert, first row, rows) per tile; row_token / row_weight per sorted
@@ -260,6 +264,7 @@ __global__ void __launch_bounds__(PLAN_THREADS) plan_kernel(const int* __restric
 
 // The choice and the plan of a step of few tokens in one block: its warps take the tokens in turn, then the
 // block sorts the pairs.  `real`: the experts that have rows (the first of the `experts` the router scores).
+template <int PL>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_plan_kernel(
     const float* __restrict__ logits, int64_t ld, int tokens, int experts, int top, int softmax,
     const float* __restrict__ correction, RoutePick rule, int* ids, float* weights, int real, int tile_rows,
@@ -267,7 +272,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) route_plan_kernel(
     int* __restrict__ pair_row, int* err) {
   ls_dependency_sync();
   for (int t = threadIdx.x >> 5; t < tokens; t += ROUTE_WARPS)
-    route_token(logits, ld, t, experts, top, softmax, correction, rule, ids, weights);
+    route_token<PL>(logits, ld, t, experts, top, softmax, correction, rule, ids, weights);
   __syncthreads();                  // (the block's own writes to ids and weights are visible to it behind the barrier)
   plan_block(ids, weights, tokens * top, top, real, tile_rows, plan, max_tiles, row_token, row_weight, pair_row, err);
 }
@@ -395,6 +400,15 @@ __global__ void __launch_bounds__(256) mix_kernel(const float* __restrict__ y, c
   }
 }
 
+// the instance whose lanes look after no more experts than there are (a choice does not depend on it)
+template <typename F>
+cudaError_t per_lane(int experts, F launch) {
+  if (experts <= 32) return launch(std::integral_constant<int, 1>());
+  if (experts <= 64) return launch(std::integral_constant<int, 2>());
+  if (experts <= 128) return launch(std::integral_constant<int, 4>());
+  return launch(std::integral_constant<int, MAX_PER_LANE>());
+}
+
 // groups 0: no limit; else equal groups, the kept ones of which hold enough experts
 bool pick_ok(int experts, int top, int groups, int keep) {
   if (groups == 0) return true;
@@ -412,8 +426,10 @@ LS_API int ls_experts_route(const float* logits, long long ld, int tokens, int e
   if (!pick_ok(experts, top, groups, keep)) return LS_E_SIZE;
   if (experts <= 0 || experts > 32 * MAX_PER_LANE || top <= 0 || top > experts || ld < experts) return LS_E_SIZE;
   LS_COUNT(LS_K_EXPERTS_ROUTE);
-  cudaError_t e = ls_launch(route_kernel, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream,
+  cudaError_t e = per_lane(experts, [&](auto pl) {
+    return ls_launch(route_kernel<decltype(pl)::value>, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream,
                             logits, (int64_t)ld, tokens, experts, top, softmax, correction, RoutePick{groups, keep, factor}, ids, weights);
+  });
   if (e != cudaSuccess) return (int)e;
   return ls_launch_status();
 }
@@ -429,9 +445,11 @@ LS_API int ls_experts_route_plan(const float* logits, long long ld, int tokens, 
   if (real <= 0 || real > experts || max_tiles <= 0 || tile_rows <= 0) return LS_E_SIZE;
   LS_COUNT(LS_K_EXPERTS_ROUTE);
   LS_COUNT(LS_K_EXPERTS_PLAN);
-  cudaError_t e = ls_launch(route_plan_kernel, dim3(1), dim3(ROUTE_WARPS * 32), sizeof(int) * 3 * (size_t)real, stream,
+  cudaError_t e = per_lane(experts, [&](auto pl) {
+    return ls_launch(route_plan_kernel<decltype(pl)::value>, dim3(1), dim3(ROUTE_WARPS * 32), sizeof(int) * 3 * (size_t)real, stream,
                             logits, (int64_t)ld, tokens, experts, top, softmax, correction, RoutePick{groups, keep, factor}, ids, weights, real, tile_rows,
                             plan, max_tiles, row_token, row_weight, pair_row, err);
+  });
   if (e != cudaSuccess) return (int)e;
   return ls_launch_status();
 }

@@ -78,73 +78,58 @@ __device__ float block_sumsq(const WideArgs& a, const T* src, int col0, int n, f
   return ls_block_sum(ss, scratch);
 }
 
-// One projection (q or k) of one token: heads of size d at src, normed, rotated, written as
-// heads of size D at dst(head) (the padding as zeros).  KEYS: `maps` of them share a row of D, side by side;
-// else (queries) each has a row of its own, its elements at its map's place.
-template <typename T, bool KEYS, typename Dst>
-__device__ void finish_heads(const WideArgs& a, const T* src, int col0, int heads, const void* gain, float rstd_whole,
-                             const float* cs, const float* sn, float* head_rstd, float factor, Dst dst) {
-  const int d = a.d, D = a.D, half = a.rot_dim >> 1;
+// One head of one token's queries or keys by one warp: d elements at src (column `col0` of the whole row), normed, rotated,
+// times `factor`, written to dst[0 .. d).  `g0`: where the head's gain begins.
+template <typename T>
+__device__ __forceinline__ void finish_head(const WideArgs& a, const T* src, int col0, const void* gain, int g0, float rstd,
+                                            const float* cs, const float* sn, float factor, T* dst) {
+  const int d = a.d, half = a.rot_dim >> 1, lane = threadIdx.x & 31;
   if (a.scope == 1 && gain != nullptr) {
-    // per-head sums: a warp per head, lanes strided, xor-tree
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int h = warp; h < heads; h += THREADS / 32) {
-      float ss = 0.f;
-      for (int i = lane; i < d; i += 32) {
-        const float v = biased_at<T>(a, src, col0, h * d + i);
-        ss = fmaf(v, v, ss);
-      }
-      ss = ls_warp_sum(ss);
-      if (lane == 0) head_rstd[h] = 1.0f / sqrtf(ss / (float)d + a.eps);
+    float ss = 0.f;
+    for (int i = lane; i < d; i += 32) {
+      const float v = biased_at<T>(a, src, col0, i);
+      ss = fmaf(v, v, ss);
     }
-    __syncthreads();
+    rstd = 1.0f / sqrtf(ls_warp_sum(ss) / (float)d + a.eps);
   }
-  const int rows = KEYS ? heads / a.maps : heads;
-  for (int e = threadIdx.x; e < rows * D; e += THREADS) {
-    const int row = e / D, at = e - row * D;
-    int h = row, i = at;                                 // the head and the element of it that lie here
-    if (a.maps > 1) {
-      const int map = at / d;
-      const bool here = map < a.maps && (KEYS || map == row % a.maps);
-      if (KEYS) h = row * a.maps + map;
-      i = here ? at - map * d : d;
-    }
-    float out = 0.f;
-    if (i < d) {
-      auto normed = [&](int j) {
-        float v = biased_at<T>(a, src, col0, h * d + j);
-        if (gain != nullptr) {
-          v = __fmul_rn(v, a.scope == 2 ? rstd_whole : head_rstd[h]);
-          v = __fmul_rn(v, gain_at(gain, a.gain_bf16, a.scope == 2 ? h * d + j : j));
-        }
-        return v;
-      };
-      if (i < a.rot_dim && a.interleaved) {
-        const int r = i >> 1;
-        const float lo = normed(2 * r), hi = normed(2 * r + 1);
-        out = (i & 1) == 0 ? __fsub_rn(__fmul_rn(lo, cs[r]), __fmul_rn(hi, sn[r]))
-                           : __fadd_rn(__fmul_rn(hi, cs[r]), __fmul_rn(lo, sn[r]));
-      } else if (i < a.rot_dim) {
-        if (i < half) {
-          const float lo = normed(i), hi = normed(i + half);
-          out = __fsub_rn(__fmul_rn(lo, cs[i]), __fmul_rn(hi, sn[i]));
-        } else {
-          const float lo = normed(i - half), hi = normed(i);
-          out = __fadd_rn(__fmul_rn(hi, cs[i - half]), __fmul_rn(lo, sn[i - half]));
-        }
+  auto normed = [&](int j) {
+    float v = biased_at<T>(a, src, col0, j);
+    if (gain != nullptr) v = __fmul_rn(__fmul_rn(v, rstd), gain_at(gain, a.gain_bf16, g0 + j));
+    return v;
+  };
+  for (int i = lane; i < d; i += 32) {
+    float out;
+    if (i < a.rot_dim && a.interleaved) {
+      const int r = i >> 1;
+      const float lo = normed(2 * r), hi = normed(2 * r + 1);
+      out = (i & 1) == 0 ? __fsub_rn(__fmul_rn(lo, cs[r]), __fmul_rn(hi, sn[r]))
+                         : __fadd_rn(__fmul_rn(hi, cs[r]), __fmul_rn(lo, sn[r]));
+    } else if (i < a.rot_dim) {
+      if (i < half) {
+        const float lo = normed(i), hi = normed(i + half);
+        out = __fsub_rn(__fmul_rn(lo, cs[i]), __fmul_rn(hi, sn[i]));
       } else {
-        out = normed(i);
+        const float lo = normed(i - half), hi = normed(i);
+        out = __fadd_rn(__fmul_rn(hi, cs[i - half]), __fmul_rn(lo, sn[i - half]));
       }
-      if (factor != 1.0f) out = __fmul_rn(out, factor);
+    } else {
+      out = normed(i);
     }
-    dst(row, at, out);
+    if (factor != 1.0f) out = __fmul_rn(out, factor);
+    dst[i] = ls_from_float<T>(out);
   }
 }
 
+// zeros in dst[from .. to), by one warp
+template <typename T>
+__device__ __forceinline__ void zero_span(T* dst, int from, int to) {
+  for (int i = from + (int)(threadIdx.x & 31); i < to; i += 32) dst[i] = ls_from_float<T>(0.f);
+}
+
+// A block per token, a warp per head of q, then of k, then of v.
 template <typename T>
 __global__ void __launch_bounds__(THREADS) qkv_finish_kernel(WideArgs a, int* err) {
   __shared__ float scratch[32];
-  __shared__ float head_rstd[256];
   ls_dependency_sync();
   const int t = blockIdx.x;
   const T* row = reinterpret_cast<const T*>(a.qkv) + (int64_t)t * a.ld;
@@ -156,48 +141,55 @@ __global__ void __launch_bounds__(THREADS) qkv_finish_kernel(WideArgs a, int* er
   }
   const float* cs = a.cos_table + (int64_t)pos * half;
   const float* sn = a.sin_table + (int64_t)pos * half;
-
-  // queries
-  float rstd = 1.f;
+  const int nk = a.nkv * a.maps;
+  const bool writes = a.has_kv && a.write_cache;
+  float q_rstd = 1.f, k_rstd = 1.f;
   if (a.scope == 2 && a.q_gain != nullptr)
-    rstd = 1.0f / sqrtf(block_sumsq<T>(a, row, 0, a.nq * a.d, scratch) / (float)(a.nq * a.d) + a.eps);
-  T* q_dst = reinterpret_cast<T*>(a.q_out) + (int64_t)t * a.nq * a.D;
+    q_rstd = 1.0f / sqrtf(block_sumsq<T>(a, row, 0, a.nq * a.d, scratch) / (float)(a.nq * a.d) + a.eps);
+  if (a.scope == 2 && a.k_gain != nullptr && writes) {
+    __syncthreads();
+    k_rstd = 1.0f / sqrtf(block_sumsq<T>(a, row + a.nq * a.d, a.nq * a.d, nk * a.d, scratch) / (float)(nk * a.d) + a.eps);
+  }
+  // where the token's keys and values go
+  int page = -1, in_page = 0;
+  if (writes) {
+    const int req = a.token_req[t];
+    page = a.block_table[(int64_t)req * a.table_stride + pos / a.page_size];
+    in_page = pos % a.page_size;
+    if (page < 0 || page >= a.num_pages) {
+      if (threadIdx.x == 0) ls_record_fault(err, LS_DEV_PAGE_RANGE, t);
+      page = -1;
+    }
+  }
   const float temperature =
       a.temp_coef != 0.f ? 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1)) : 1.0f;
-  finish_heads<T, false>(a, row, 0, a.nq, a.q_gain, rstd, cs, sn, head_rstd, temperature,
-                  [&](int h, int i, float v) { q_dst[h * a.D + i] = ls_from_float<T>(v); });
-  if (!a.has_kv || !a.write_cache) return;
-
-  // keys and values into the token's page
-  const int req = a.token_req[t];
-  const int page = a.block_table[(int64_t)req * a.table_stride + pos / a.page_size];
-  if (page < 0 || page >= a.num_pages) {
-    if (threadIdx.x == 0) ls_record_fault(err, LS_DEV_PAGE_RANGE, t);
-    return;
-  }
-  const int in_page = pos % a.page_size;
-  T* pages = reinterpret_cast<T*>(a.pages);
-  const T* k_src = row + a.nq * a.d;
-  const T* v_src = k_src + a.nkv * a.maps * a.d;
-  float k_rstd = 1.f;
-  if (a.scope == 2 && a.k_gain != nullptr) {
-    __syncthreads();
-    k_rstd = 1.0f / sqrtf(block_sumsq<T>(a, k_src, a.nq * a.d, a.nkv * a.maps * a.d, scratch) / (float)(a.nkv * a.maps * a.d) + a.eps);
-  }
-  __syncthreads();          // head_rstd is used again
-  finish_heads<T, true>(a, k_src, a.nq * a.d, a.nkv * a.maps, a.k_gain, k_rstd, cs, sn, head_rstd, 1.0f, [&](int h, int i, float v) {
-    pages[((((int64_t)page * 2 + 0) * a.nkv + h) * a.page_size + in_page) * a.D + i] = ls_from_float<T>(v);
-  });
   const T* other = a.v_other != nullptr ? reinterpret_cast<const T*>(a.v_other) + (int64_t)t * a.v_other_ld : nullptr;
-  const float mix = other != nullptr ? *a.v_mix : 0.f;
-  for (int e = threadIdx.x; e < a.nkv * a.D; e += THREADS) {
-    const int h = e / a.D, i = e - h * a.D;
-    float v = 0.f;
-    if (i < a.dv) {
-      v = biased_at<T>(a, v_src, (a.nq + a.nkv * a.maps) * a.d, h * a.dv + i);
-      if (other != nullptr) v = __fadd_rn(__fmul_rn(1.0f - mix, v), __fmul_rn(mix, ls_to_float<T>(other[h * a.dv + i])));
+  const float mix = other != nullptr && page >= 0 ? *a.v_mix : 0.f;
+  T* pages = reinterpret_cast<T*>(a.pages);
+  const int tasks = a.nq + (page >= 0 ? nk + a.nkv : 0);
+  for (int task = threadIdx.x >> 5; task < tasks; task += THREADS / 32) {
+    if (task < a.nq) {
+      // a query sub-head lies where its map's key lies, between zeros
+      T* dst = reinterpret_cast<T*>(a.q_out) + ((int64_t)t * a.nq + task) * a.D;
+      const int at = (task % a.maps) * a.d;
+      finish_head<T>(a, row + task * a.d, task * a.d, a.q_gain, a.scope == 2 ? task * a.d : 0, q_rstd, cs, sn, temperature, dst + at);
+      zero_span<T>(dst, 0, at);
+      zero_span<T>(dst, at + a.d, a.D);
+    } else if (task < a.nq + nk) {
+      const int h = task - a.nq, slot = h / a.maps, map = h - slot * a.maps, col = task * a.d;
+      T* dst = pages + ((((int64_t)page * 2 + 0) * a.nkv + slot) * a.page_size + in_page) * a.D;
+      finish_head<T>(a, row + col, col, a.k_gain, a.scope == 2 ? h * a.d : 0, k_rstd, cs, sn, 1.0f, dst + map * a.d);
+      if (map == a.maps - 1) zero_span<T>(dst, a.maps * a.d, a.D);
+    } else {
+      const int h = task - a.nq - nk, col = (a.nq + nk) * a.d;
+      T* dst = pages + ((((int64_t)page * 2 + 1) * a.nkv + h) * a.page_size + in_page) * a.D;
+      for (int i = threadIdx.x & 31; i < a.dv; i += 32) {
+        float v = biased_at<T>(a, row + col, col, h * a.dv + i);
+        if (other != nullptr) v = __fadd_rn(__fmul_rn(1.0f - mix, v), __fmul_rn(mix, ls_to_float<T>(other[h * a.dv + i])));
+        dst[i] = ls_from_float<T>(v);
+      }
+      zero_span<T>(dst, a.dv, a.D);
     }
-    pages[((((int64_t)page * 2 + 1) * a.nkv + h) * a.page_size + in_page) * a.D + i] = ls_from_float<T>(v);
   }
 }
 
@@ -326,7 +318,6 @@ LS_API int ls_qkv_finish(const void* qkv, int64_t ld, void* q_out, void* pages, 
   if (nq <= 0 || nkv <= 0 || d <= 0 || dv <= 0 || maps < 1 || D < (int64_t)maps * d || D < dv || scope < 0 || scope > 2 || nq % maps)
     return LS_E_SIZE;
   if (rot_dim < 0 || rot_dim > d || (rot_dim & 1)) return LS_E_SIZE;
-  if (scope == 1 && (nq > 256 || (int64_t)nkv * maps > 256)) return LS_E_SIZE;
   if (gain_dtype != LS_F32 && gain_dtype != LS_BF16) return LS_E_DTYPE;
   if (write_cache && (pages == nullptr || page_size <= 0)) return LS_E_SIZE;
   if (temp_coef != 0.f && temp_every <= 0) return LS_E_SIZE;

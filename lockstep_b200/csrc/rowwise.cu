@@ -159,6 +159,58 @@ norm_merge_add_kernel(float* __restrict__ residual, const float* __restrict__ br
   }
 }
 
+// The same for one result without a norm of its own (n = 1, no branch gain, scale 1) and rows of up to KEEP x 256
+// elements: the row stays in registers, sums and roundings are those of norm_merge_add_kernel.
+template <int KEEP, typename TO>
+__global__ void __launch_bounds__(ROW_THREADS)
+norm_add_kernel(float* __restrict__ residual, const float* __restrict__ x, const float* __restrict__ post_gain,
+                const float* __restrict__ post_bias, const float* __restrict__ next_gain, const float* __restrict__ next_bias,
+                TO* __restrict__ next_out, int width, float eps_post, float eps_next) {
+  __shared__ float scratch[32];
+  ls_dependency_sync();
+  const int r = blockIdx.x, tid = threadIdx.x;
+  const float* row = x + (int64_t)r * width;
+  float* dst = residual + (int64_t)r * width;
+  float v[KEEP], h[KEEP];
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) v[j] = tid + j * ROW_THREADS < width ? row[tid + j * ROW_THREADS] : 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) h[j] = tid + j * ROW_THREADS < width ? dst[tid + j * ROW_THREADS] : 0.f;
+  auto moments = [&](const float (&u)[KEEP], float eps, float& mean, float& rstd) {
+    float s = 0.f, q = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) s += u[j];
+    mean = row_sum(s, scratch) / (float)width;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      const float d = tid + j * ROW_THREADS < width ? u[j] - mean : 0.f;
+      q = fmaf(d, d, q);
+    }
+    rstd = 1.0f / sqrtf(row_sum(q, scratch) / (float)width + eps);
+  };
+  float mean, rstd;
+  moments(v, eps_post, mean, rstd);
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int i = tid + j * ROW_THREADS;
+    if (i < width) {
+      const float u = (v[j] - mean) * rstd;
+      dst[i] = h[j] = h[j] + scaled(u, post_gain[i], post_bias != nullptr, post_bias != nullptr ? post_bias[i] : 0.f);
+    }
+  }
+  if (next_gain == nullptr) return;
+  moments(h, eps_next, mean, rstd);
+  TO* to = next_out + (int64_t)r * width;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int i = tid + j * ROW_THREADS;
+    if (i < width) {
+      const float u = (h[j] - mean) * rstd;
+      to[i] = ls_from_float<TO>(scaled(u, next_gain[i], next_bias != nullptr, next_bias != nullptr ? next_bias[i] : 0.f));
+    }
+  }
+}
+
 // out[t] = table[id] factor + pairs[row(previous id, id)]
 template <typename T>
 __global__ void pair_embed_kernel(const int* __restrict__ ids, const int* __restrict__ token_slot,
@@ -350,6 +402,21 @@ LS_API int ls_norm_merge_add(float* residual, const float* branches, int n, long
   }
   if (next_gain != nullptr) LS_COUNT(LS_K_NORM_MERGE_NORM);
   else LS_COUNT(LS_K_NORM_MERGE_ADD);
+  if (n == 1 && branch_gain == nullptr && scale == 1.0f && post_gain != nullptr && width <= 8 * ROW_THREADS) {
+#define LS_NA(KEEP, TO)                                                                                                  \
+  ls_launch(norm_add_kernel<KEEP, TO>, dim3(rows), dim3(ROW_THREADS), 0, stream, residual, branches, post_gain, post_bias, \
+            next_gain, next_bias, (TO*)next_out, width, eps_post, eps_next)
+    const bool f32 = next_gain == nullptr || next_dtype == LS_F32;
+    if (width <= 4 * ROW_THREADS) {
+      if (f32) LS_NA(4, float);
+      else LS_NA(4, __nv_bfloat16);
+    } else {
+      if (f32) LS_NA(8, float);
+      else LS_NA(8, __nv_bfloat16);
+    }
+#undef LS_NA
+    return ls_launch_status();
+  }
 #define LS_NM(TO)                                                                                                       \
   ls_launch(norm_merge_add_kernel<TO>, dim3(rows), dim3(ROW_THREADS), smem, stream, residual, branches, n,              \
             (int64_t)branch_stride, branch_gain, scale, post_gain, post_bias, next_gain, next_bias, (TO*)next_out, rows, \
