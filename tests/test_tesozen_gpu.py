@@ -201,7 +201,7 @@ def _fake_step(starts_and_lengths, page, nkv, d, dtype, chunk, gen):
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("page", [8, 16, 64])
-@pytest.mark.parametrize("heads, kv, d, dv", [(4, 2, 32, 64), (2, 2, 64, 128), (3, 1, 20, 30)])
+@pytest.mark.parametrize("heads, kv, d, dv", [(6, 2, 32, 64), (2, 2, 64, 128), (3, 1, 20, 30)])
 @pytest.mark.parametrize("chunk", [1, 7, 64, 100, 300, 0])
 def test_differential_attention_in_chunks(dtype, page, heads, kv, d, dv, chunk):
     """Portions and single tokens at a chunk's first and last positions, across its edge and far on, against the plain maps
@@ -293,7 +293,7 @@ def test_per_head_products_with_a_gate(dtype, tokens, heads, n, k):
 
 
 @pytest.mark.parametrize("experts, top, groups, scale", [
-    (8, 3, (4, 3), 1.5), (6, 2, (3, 1), 1.0), (1, 1, (1, 1), 2.0), (5, 5, None, 0.7), (32, 4, (8, 4), 2.5), (40, 6, (10, 5), 1.0),
+    (12, 3, (4, 3), 1.4), (6, 2, (3, 1), 1.0), (1, 1, (1, 1), 2.0), (5, 5, None, 0.7), (32, 4, (8, 4), 2.5), (40, 6, (10, 5), 1.0),
     (64, 8, (64, 9), 1.0), (96, 4, (2, 1), 3.0), (300, 7, (60, 13), 1.0), (512, 16, (8, 4), 2.5)])
 def test_choice_among_the_best_groups(experts, top, groups, scale):
     """Both kernels of the choice (one that also plans, for few tokens), with negative choice scores and corrections that change
